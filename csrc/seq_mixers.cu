@@ -23,30 +23,11 @@
 //   channel_decay_gates   decay per (head, key channel) pair for linear_recurrence (its per-channel form), sigmoid write strength
 //   sigmoid_gate_rows, power_norm_act   sigmoid gate per channel or per head in place; p1 z/rms(z) + p2 z^2/rms(z^2) + p3 z^3/rms(z^3) + p0
 #include <algorithm>
-#include "sxb_common.cuh"
+#include "seq_common.cuh"
 #include <cuda_pipeline.h>
 
 namespace sxb {
 namespace seqmix {
-
-
-
-#define SEQMIX_DISPATCH(dtype, ...)                \
-  do {                                             \
-    if ((dtype) == 0) {                         \
-      using T = float;                             \
-      __VA_ARGS__;                                 \
-    } else if ((dtype) == 2) {                 \
-      using T = __nv_bfloat16;                     \
-      __VA_ARGS__;                                 \
-    } else {                                       \
-      return SXB_ERR_UNSUPPORTED;                  \
-    }                                              \
-  } while (0)
-
-__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
-__device__ __forceinline__ float softplus_f(float x) { return x > 30.f ? x : log1pf(expf(x)); }
-__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 
 // ------------------------------------------------------------------------------------------------ embedding
 template <typename T>
@@ -307,20 +288,6 @@ constexpr int kMaxVPerLane = 8;      // value head size <= 256
 constexpr int kShortAtom = 16;       // atoms of at most this many queries run one warp per (query, head)
 constexpr int kBQ = 64, kBK = 64;    // query rows / keys per tile of the tiled kernel
 
-template <typename T>
-__device__ __forceinline__ float4 load4_f32(const T* p);
-template <>
-__device__ __forceinline__ float4 load4_f32<float>(const float* p) {
-  return *reinterpret_cast<const float4*>(p);
-}
-template <>
-__device__ __forceinline__ float4 load4_f32<__nv_bfloat16>(const __nv_bfloat16* p) {
-  const uint2 u = *reinterpret_cast<const uint2*>(p);
-  const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(&u.x);
-  const __nv_bfloat162 b = *reinterpret_cast<const __nv_bfloat162*>(&u.y);
-  return make_float4(__low2float(a), __high2float(a), __low2float(b), __high2float(b));
-}
-
 // Tiled form for atoms of many queries (prompt portions): one CTA per (64 queries of an atom, query head).  Q (scaled),
 // one 64-key tile of K and V (converted to fp32) and the tile's weights (in the key tile's place, once the scores are
 // done: head sizes up to 128 then leave room for two CTAs per SM) sit in shared memory; 256 threads hold 4x4
@@ -333,7 +300,7 @@ sink_attention_tile_kernel(const float* __restrict__ q, const T* __restrict__ kc
                            const int* __restrict__ tables, int max_blocks, int block_size, int Hq, int G, int d,
                            int dv, float scale, int chunk, int window, int kpitch, int vpitch,
                            const float* __restrict__ dist_bias, int bias_len, const T* __restrict__ gate,
-                           long long gate_ld) {
+                           long long gate_ld, int gate_heads) {
   extern __shared__ __align__(16) float smf[];
   const int dp = d + 4, vp = NV * 64, pp = kBK + 4;
   float* Qs = smf;
@@ -479,7 +446,7 @@ sink_attention_tile_kernel(const float* __restrict__ q, const T* __restrict__ kc
         const float2 a2 = acc[i][n * 2 + (e >> 1)];
         if (c < dv) {
           float o = ((e & 1) ? a2.y : a2.x) * inv;
-          if (gate != nullptr) o *= sigmoid_f(to_f32<T>(gate[(long long)(row0 + r) * gate_ld + h * dv + c]));
+          if (gate != nullptr) o *= sigmoid_f(to_f32<T>(gate[(long long)(row0 + r) * gate_ld + (gate_heads ? h : h * dv + c)]));
           out[((long long)(row0 + r) * Hq + h) * dv + c] = from_f32<T>(o);
         }
       }
@@ -521,7 +488,7 @@ sink_attention_kernel(const float* __restrict__ q, const T* __restrict__ kcache,
                       const int* __restrict__ tok_pos, const int* __restrict__ tables, int max_blocks, int block_size,
                       int Hq, int G, int d, int dv, float scale, int chunk, int window, int kpitch, int vpitch,
                       const int* __restrict__ atoms, const float* __restrict__ dist_bias, int bias_len,
-                      const T* __restrict__ gate, long long gate_ld) {
+                      const T* __restrict__ gate, long long gate_ld, int gate_heads) {
   // q [REP][d8] | partial values [kAW][REP][dv] | partial max [kAW][REP] | partial sum [kAW][REP] | key staging
   extern __shared__ __align__(16) float qs[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -680,7 +647,7 @@ sink_attention_kernel(const float* __restrict__ q, const T* __restrict__ kcache,
       o += pacc[(w * REP + hh) * dv + c] * f;
     }
     float r = L > 0.f ? o / L : 0.f;
-    if (gate != nullptr) r *= sigmoid_f(to_f32<T>(gate[(long long)t * gate_ld + (h0 + hh) * dv + c]));
+    if (gate != nullptr) r *= sigmoid_f(to_f32<T>(gate[(long long)t * gate_ld + (gate_heads ? h0 + hh : (h0 + hh) * dv + c)]));
     out[((long long)t * Hq + h0 + hh) * dv + c] = from_f32<T>(r);
   }
 }
@@ -690,7 +657,7 @@ static int launch_attention_rows_v(dim3 grid, const void* q, const void* kcache,
                                    void* out, const void* tok_seq, const void* tok_pos, const void* tables,
                                    int max_blocks, int block_size, int Hq, int G, int d, int dv, float scale,
                                    int chunk, int window, int kpitch, int vpitch, const int* atoms, const void* dist_bias,
-                                   int bias_len, const void* gate, long long gate_ld, cudaStream_t s) {
+                                   int bias_len, const void* gate, long long gate_ld, int gate_heads, cudaStream_t s) {
   const size_t smem = (size_t)(REP * ((d + 7) & ~7) + kAW * REP * dv + 2 * kAW * REP + kAW * 32 * 68) * sizeof(float);
   cudaError_t e = cudaFuncSetAttribute(sink_attention_kernel<T, REP, VPL>,
                                        cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -699,7 +666,7 @@ static int launch_attention_rows_v(dim3 grid, const void* q, const void* kcache,
   sink_attention_kernel<T, REP, VPL><<<grid, 32 * kAW, smem, s>>>(
       (const float*)q, (const T*)kcache, (const T*)vcache, (const float*)sink, (T*)out, (const int*)tok_seq,
       (const int*)tok_pos, (const int*)tables, max_blocks, block_size, Hq, G, d, dv, scale, chunk, window, kpitch,
-      vpitch, atoms, (const float*)dist_bias, bias_len, (const T*)gate, gate_ld);
+      vpitch, atoms, (const float*)dist_bias, bias_len, (const T*)gate, gate_ld, gate_heads);
   return SXB_OK;
 }
 
@@ -708,14 +675,14 @@ static int launch_attention_rows(dim3 grid, const void* q, const void* kcache, c
                                  void* out, const void* tok_seq, const void* tok_pos, const void* tables,
                                  int max_blocks, int block_size, int Hq, int G, int d, int dv, float scale, int chunk,
                                  int window, int kpitch, int vpitch, const int* atoms, const void* dist_bias,
-                                 int bias_len, const void* gate, long long gate_ld, cudaStream_t s) {
+                                 int bias_len, const void* gate, long long gate_ld, int gate_heads, cudaStream_t s) {
   if (dv <= 128)
     return launch_attention_rows_v<T, REP, 4>(grid, q, kcache, vcache, sink, out, tok_seq, tok_pos, tables, max_blocks,
                                               block_size, Hq, G, d, dv, scale, chunk, window, kpitch, vpitch, atoms,
-                                              dist_bias, bias_len, gate, gate_ld, s);
+                                              dist_bias, bias_len, gate, gate_ld, gate_heads, s);
   return launch_attention_rows_v<T, REP, kMaxVPerLane>(grid, q, kcache, vcache, sink, out, tok_seq, tok_pos, tables,
                                                        max_blocks, block_size, Hq, G, d, dv, scale, chunk, window,
-                                                       kpitch, vpitch, atoms, dist_bias, bias_len, gate, gate_ld, s);
+                                                       kpitch, vpitch, atoms, dist_bias, bias_len, gate, gate_ld, gate_heads, s);
 }
 
 // Query heads per key/value head that one CTA takes together: the largest of 8, 4, 2, 1 that divides the group.
@@ -723,7 +690,7 @@ static int attention_rows(int dtype, dim3 grid, const void* q, const void* kcach
                           const void* sink, void* out, const void* tok_seq, const void* tok_pos, const void* tables,
                           int max_blocks, int block_size, int Hq, int G, int d, int dv, float scale, int chunk,
                           int window, int kpitch, int vpitch, const int* atoms, const void* dist_bias, int bias_len,
-                          const void* gate, long long gate_ld, cudaStream_t s) {
+                          const void* gate, long long gate_ld, int gate_heads, cudaStream_t s) {
   const int group = Hq / G;
   int rc = SXB_OK;
   // (Taking fewer heads together when a decode batch leaves SMs idle was measured slower: every CTA walks all keys.)
@@ -732,7 +699,7 @@ static int attention_rows(int dtype, dim3 grid, const void* q, const void* kcach
   SEQMIX_DISPATCH(dtype, (rc = launch_attention_rows<T, REP>(grid, q, kcache, vcache, sink, out, tok_seq, tok_pos,      \
                                                               tables, max_blocks, block_size, Hq, G, d, dv, scale,      \
                                                               chunk, window, kpitch, vpitch, atoms, dist_bias,      \
-                                                              bias_len, gate, gate_ld, s)))
+                                                              bias_len, gate, gate_ld, gate_heads, s)))
   if (rep == 8) ROWS(8);
   else if (rep == 4) ROWS(4);
   else if (rep == 2) ROWS(2);
@@ -773,21 +740,6 @@ conv_silu_kernel(const T* __restrict__ x, long long ld, const T* __restrict__ w,
 // is loaded by the rule above at the thread's first row and at a sequence's first row in the batch, and shifted
 // otherwise; the sum runs in the same order as in the scalar kernel.
 constexpr int kConvRows = 8;
-
-template <typename T>
-__device__ __forceinline__ void load8_f32(const T* p, float* o);
-template <>
-__device__ __forceinline__ void load8_f32<float>(const float* p, float* o) {
-  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-  o[0] = a.x, o[1] = a.y, o[2] = a.z, o[3] = a.w, o[4] = b.x, o[5] = b.y, o[6] = b.z, o[7] = b.w;
-}
-template <>
-__device__ __forceinline__ void load8_f32<__nv_bfloat16>(const __nv_bfloat16* p, float* o) {
-  const uint4 u = *reinterpret_cast<const uint4*>(p);
-  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
-#pragma unroll
-  for (int i = 0; i < 4; ++i) o[2 * i] = __low2float(h[i]), o[2 * i + 1] = __high2float(h[i]);
-}
 
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128)
@@ -1629,20 +1581,20 @@ SXB_API int sxb_qkv_filter_norm_append(const void* qkv, long long ld, const void
  * vcache + slot * v_pitch + g * dv (pitches in elements; 0 = packed [pages, block_size, G, d|dv]), so values may be a
  * column range of the key rows.  out `dtype` [n_tokens, Hq * dv] (the caches have the same type).  dist_bias (fp32
  * [Hq, bias_len] or null) is added to the scaled score of a key at distance n = query position - key position:
- * dist_bias[h, min(n, bias_len - 1)].  gate (`dtype` rows of pitch gate_ld with Hq * dv channels, or null): the output is
- * multiplied by sigmoid(gate).  One CTA per (token, head group). */
+ * dist_bias[h, min(n, bias_len - 1)].  gate (`dtype` rows of pitch gate_ld with Hq * dv channels, or Hq when
+ * gate_heads != 0, or null): the output is multiplied by sigmoid(gate), per channel or per head.  One CTA per (token, head group). */
 SXB_API int sxb_sink_attention(const void* q, const void* kcache, const void* vcache, const void* sink, void* out,
                                const void* tok_seq, const void* tok_pos, const void* tables, int n_tokens,
                                int max_blocks, int block_size, int Hq, int G, int d, int dv, float scale, int chunk,
                                int window, int k_pitch, int v_pitch, const void* dist_bias, int bias_len,
-                               const void* gate, long long gate_ld, int dtype, void* stream) {
+                               const void* gate, long long gate_ld, int gate_heads, int dtype, void* stream) {
   if (n_tokens <= 0) return SXB_OK;
   if (dv > 32 * kMaxVPerLane || Hq % G || (dist_bias != nullptr && bias_len < 1)) return SXB_ERR_UNSUPPORTED;
   if (k_pitch <= 0) k_pitch = G * d;
   if (v_pitch <= 0) v_pitch = G * dv;
   const int rc = attention_rows(dtype, dim3(n_tokens, 1), q, kcache, vcache, sink, out, tok_seq, tok_pos, tables,
                                 max_blocks, block_size, Hq, G, d, dv, scale, chunk, window, k_pitch, v_pitch, nullptr,
-                                dist_bias, bias_len, gate, gate_ld, (cudaStream_t)stream);
+                                dist_bias, bias_len, gate, gate_ld, gate_heads, (cudaStream_t)stream);
   if (rc != SXB_OK) return rc;
   SXB_CHECK_LAUNCH();
   return SXB_OK;
@@ -1763,7 +1715,7 @@ static int launch_attention_tiles(const void* q, const void* kcache, const void*
                                   const void* atoms, int n_long, const void* tables, int max_blocks, int block_size,
                                   int Hq, int G, int d, int dv, float scale, int chunk, int window, int kpitch,
                                   int vpitch, const void* dist_bias, int bias_len, const void* gate,
-                                  long long gate_ld, cudaStream_t s) {
+                                  long long gate_ld, int gate_heads, cudaStream_t s) {
   const size_t smem = (size_t)(kBQ * (d + 4) + std::max(kBK * (d + 4), kBQ * (kBK + 4)) + kBK * NV * 64) * sizeof(float);
   cudaError_t e = cudaFuncSetAttribute(sink_attention_tile_kernel<T, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                        (int)smem);
@@ -1771,7 +1723,7 @@ static int launch_attention_tiles(const void* q, const void* kcache, const void*
   sink_attention_tile_kernel<T, NV><<<dim3(2 * n_long, Hq), 256, smem, s>>>(
       (const float*)q, (const T*)kcache, (const T*)vcache, (const float*)sink, (T*)out, (const int*)atoms,
       (const int*)tables, max_blocks, block_size, Hq, G, d, dv, scale, chunk, window, kpitch, vpitch,
-      (const float*)dist_bias, bias_len, (const T*)gate, gate_ld);
+      (const float*)dist_bias, bias_len, (const T*)gate, gate_ld, gate_heads);
   return SXB_OK;
 }
 
@@ -1782,7 +1734,7 @@ SXB_API int sxb_sink_attention_atoms(const void* q, const void* kcache, const vo
                                      const void* atoms, int n_atoms, int n_long, const void* tables, int max_blocks,
                                      int block_size, int Hq, int G, int d, int dv, float scale, int chunk, int window,
                                      int k_pitch, int v_pitch, const void* dist_bias, int bias_len, const void* gate,
-                                     long long gate_ld, int dtype, void* stream) {
+                                     long long gate_ld, int gate_heads, int dtype, void* stream) {
   if (n_atoms <= 0) return SXB_OK;
   if (dist_bias != nullptr && bias_len < 1) return SXB_ERR_UNSUPPORTED;
   if (k_pitch <= 0) k_pitch = G * d;
@@ -1797,7 +1749,7 @@ SXB_API int sxb_sink_attention_atoms(const void* q, const void* kcache, const vo
   SEQMIX_DISPATCH(dtype, (rc = launch_attention_tiles<T, NV>(q, kcache, vcache, sink, out, atoms, n_long, tables,      \
                                                               max_blocks, block_size, Hq, G, d, dv, scale, chunk,      \
                                                               window, k_pitch, v_pitch, dist_bias, bias_len, gate,     \
-                                                              gate_ld, s)))
+                                                              gate_ld, gate_heads, s)))
     if (nv == 1) TILES(1);
     else if (nv == 2) TILES(2);
     else if (nv == 3) TILES(3);
@@ -1809,7 +1761,7 @@ SXB_API int sxb_sink_attention_atoms(const void* q, const void* kcache, const vo
   if (n_atoms > n_long) {
     const int rc = attention_rows(dtype, dim3((n_atoms - n_long) * kShortAtom, 1), q, kcache, vcache, sink, out, nullptr,
                                   nullptr, tables, max_blocks, block_size, Hq, G, d, dv, scale, chunk, window, k_pitch,
-                                  v_pitch, (const int*)atoms + 6 * n_long, dist_bias, bias_len, gate, gate_ld, s);
+                                  v_pitch, (const int*)atoms + 6 * n_long, dist_bias, bias_len, gate, gate_ld, gate_heads, s);
     if (rc != SXB_OK) return rc;
     SXB_CHECK_LAUNCH();
   }

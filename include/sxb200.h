@@ -460,7 +460,7 @@ int sxb_sink_attention(const void* q, const void* kcache, const void* vcache, co
                        const void* tok_seq, const void* tok_pos, const void* tables, int n_tokens, int max_blocks,
                        int block_size, int Hq, int G, int d, int dv, float scale, int chunk, int window,
                        int k_pitch, int v_pitch, const void* dist_bias, int bias_len, const void* gate,
-                       long long gate_ld, int dtype, void* stream);
+                       long long gate_ld, int gate_heads, int dtype, void* stream);
 int sxb_conv_silu(const void* x, long long ld, const void* w, const void* bias, const void* state,
                   const void* seq_info, const void* tok_seq, void* out, int n_tokens, int C, int taps, int dtype,
                   void* stream);
@@ -485,7 +485,7 @@ int sxb_sink_attention_atoms(const void* q, const void* kcache, const void* vcac
                              const void* atoms, int n_atoms, int n_long, const void* tables, int max_blocks,
                              int block_size, int Hq, int G, int d, int dv, float scale, int chunk, int window,
                              int k_pitch, int v_pitch, const void* dist_bias, int bias_len, const void* gate,
-                             long long gate_ld, int dtype, void* stream);
+                             long long gate_ld, int gate_heads, int dtype, void* stream);
 
 /* ---- csrc/moe_ragged.cu */
 /* As sxb_moe_scatter with every copied row multiplied by its routing weight: moe_input[slot(t, k)] = x[t] * scores[t, k].
@@ -557,6 +557,25 @@ int sxb_sigmoid_gate_rows(void* x, const void* gate, long long ldg, long long ro
                           int dtype, void* stream);
 int sxb_power_norm_act(const void* in, const void* bias, const void* coef, void* out, long long rows, int F,
                        float eps, int dtype, void* stream);
+
+/* ---- csrc/parallel_mixers.cu */
+int sxb_resid_sum_step(void* resid, const void* y, const void* a, const void* wa, const void* b, const void* wb,
+                       float mult, float eps, void* rstd, const void* rows, const void* w1, void* out,
+                       const void* w2, void* out2, const void* filt, void* state, const void* seq_info,
+                       const void* tok_seq, int taps, int n_rows, int width, int dtype, void* stream);
+int sxb_norm_filter_rows(const void* x, const void* rstd, const void* w1, const void* filt, void* state,
+                         const void* seq_info, const void* tok_seq, void* out, const void* w2, void* out2,
+                         int n_tokens, int n_seqs, int width, int taps, int dtype, void* stream);
+int sxb_rope_append(const void* proj, long long ld, int q0, int k0, int v0, const void* q_w, const void* k_w,
+                    const void* inv_freq, const void* q_scale, void* q_out, void* kcache, void* vcache,
+                    const void* tok_seq, const void* tok_pos, const void* tables, int n_tokens, int max_blocks,
+                    int block_size, int Hq, int G, int d, int dv, int n_rot, int interleaved, float eps, int dtype,
+                    void* stream);
+int sxb_removal_prepare(const void* proj, long long ld, int r0, int k0, int v0, int a0, int low0, const void* w2,
+                        const void* w0, const void* a_bias, void* buf, int n_tokens, int H, int n, int rank,
+                        float rate, float eps, int dtype, void* stream);
+int sxb_removal_recurrence(const void* buf, void* state, void* out, const void* seq_info, int n_seqs, int H, int n,
+                           int single_rows, void* stream);
 
 #ifdef __cplusplus
 }

@@ -21,8 +21,8 @@ _lib.register({
     "sxb_resid_norm_step": "pppppp" "l" "i" "ff" "i" "p" "f" "p",
     "sxb_qk_norm_append": "p" "l" "ppppppp" "iiiiiii" "f" "ii" "p",
     "sxb_qkv_filter_norm_append": "p" "l" "ppppppppppp" "iiiiiiii" "f" "i" "f" "i" "i" "p",
-    "sxb_sink_attention": "pppppppp" "iiiiiii" "f" "iiii" "p" "i" "p" "l" "i" "p",
-    "sxb_sink_attention_atoms": "pppppp" "ii" "p" "iiiiii" "f" "iiii" "p" "i" "p" "l" "i" "p",
+    "sxb_sink_attention": "pppppppp" "iiiiiii" "f" "iiii" "p" "i" "p" "l" "ii" "p",
+    "sxb_sink_attention_atoms": "pppppp" "ii" "p" "iiiiii" "f" "iiii" "p" "i" "p" "l" "ii" "p",
     "sxb_conv_silu": "p" "l" "pppppp" "iii" "i" "p",
     "sxb_conv_state_update": "p" "l" "pp" "iii" "i" "p",
     "sxb_unit_norm_heads": "p" "l" "iii" "ff" "i" "p",
@@ -222,7 +222,8 @@ def sink_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, 
     latent itself.
 
     ``dist_bias`` (fp32 ``[Hq, L]``): ``dist_bias[h, min(pos - j, L - 1)]`` is added to the scaled score of key ``j``.
-    ``gate`` (``[T, Hq * dv]``, a column slice is fine): the result is multiplied by ``sigmoid(gate)``.
+    ``gate`` (``[T, Hq * dv]``, or ``[T, Hq]`` for one per head; a column slice is fine): the result is multiplied by
+    ``sigmoid(gate)``.
 
     With the batch's attention ``atoms`` (longest first) of which the first ``n_long`` hold more than
     :data:`SHORT_ATOM` queries, those run the tiled kernel (64 queries per CTA, K/V tiles shared by them) and the rest
@@ -247,8 +248,11 @@ def sink_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, 
             raise ValueError("the distance bias is a contiguous fp32 [heads, distances] table")
         if gate is not None and gate.dtype != out_dtype:
             raise ValueError("the gate has the activation dtype")
+        if gate is not None and gate.shape[1] not in (Hq, Hq * dv):
+            raise ValueError("the gate has one column per head or per output channel")
         extra = (_lib.ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[1],
-                 None if gate is None else _rows(gate).data_ptr(), 0 if gate is None else gate.stride(0))
+                 None if gate is None else _rows(gate).data_ptr(), 0 if gate is None else gate.stride(0),
+                 int(gate is not None and gate.shape[1] == Hq))
         if atoms is not None and n_long > 0 and tiles_supported(d, dv):
             _lib.call("sxb_sink_attention_atoms", q.data_ptr(), kcache.data_ptr(), vptr, _lib.ptr(sink),
                       out.data_ptr(), atoms.data_ptr(), atoms.shape[0], int(n_long), tables.data_ptr(), tables.shape[1],
@@ -281,7 +285,7 @@ def sink_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, 
         out[t] = torch.einsum("hn,nhd->hd", p, v)
     out = out.reshape(T, Hq * dv)
     if gate is not None:
-        out = out * torch.sigmoid(gate.float())
+        out = out * torch.sigmoid(gate.float()).repeat_interleave(Hq * dv // gate.shape[1], dim=1)
     return out.to(out_dtype)
 
 

@@ -1,14 +1,14 @@
 """Ragged-batch model for hybrid layer stacks: every layer names its own token mixer — attention over the paged cache
 (per-head keys and values, or one latent vector per token), a gated-delta-rule (one decay per head, or per head and
-key channel), state-space-duality or matrix-memory LSTM recurrence — and may or may not have a feed-forward (gated,
-biased, or a mixture of experts); a span of layers can be executed several times in a row with the same weights, and
+key channel, or separate decay and removal vectors), state-space-duality or matrix-memory LSTM recurrence, or two of these side
+by side — and may or may not have a feed-forward (gated, biased, or a mixture of experts); a span of layers can be executed several times in a row with the same weights, and
 single layers can borrow another layer's weights, every execution with its own cache or state.
 
 The stack is data (:class:`HybridSpec`), as :class:`~.inference_transformer_base.ArchSpec` is for the uniform
 transformer family; per-architecture policies (``fomalix/policy.py``) fill it from a checkpoint's configuration and fuse
 the checkpoint's tensors into the projection layouts the mixer modules declare.
 
-Three layer forms (``HybridSpec.block_form``).  ``"sandwich"``: ``x += post_norm(sublayer(pre_norm(x)))``.
+Four layer forms (``HybridSpec.block_form``).  ``"sandwich"``: ``x += post_norm(sublayer(pre_norm(x)))``.
 ``"pre_scaled"``: ``x += m * sublayer(pre_norm(x))`` with one multiplier ``m`` for the whole stack (with ``layer_scale``
 also a learned scale per layer, sublayer and channel: ``x += m * ls (.) sublayer(pre_norm(x))``; with
 ``norm_weight_offset`` the norms multiply by ``offset + w``), and optionally a
@@ -18,6 +18,8 @@ part of one more embedding row of the token (``token_side_dim`` channels per lay
 per-channel scale, a short causal filter with a skip path in front of every sublayer (its last inputs are state of the
 sequence), and optionally the stream handed to the next layer is a learned mixture of the embedding and of all
 layers' results so far (``depth_mix``).
+``"parallel"``: ``x += mixer(c(norm1(x))) + ff(norm2(x))``, both of the same ``x``, with ``c(h) = h + filter(h)`` (the filter's last
+inputs are state of the sequence); a repeated span adds nothing between its passes.
 
 Numerics: the residual stream, norms, softmax, recurrences and their gates are fp32; projections, short convolutions'
 inputs, the KV cache and the sublayer outputs use ``spec.dtype`` (bf16 when serving; fp32 evaluates everything in
@@ -36,6 +38,7 @@ from ....ops import functional as F
 from ..config_v2 import RaggedInferenceEngineConfig
 from ..inference_utils import ActivationType, DtypeEnum, NormTypeEnum, ceil_div
 from ..kernels import mixer_ops as M
+from ..kernels import parallel_ops as P
 from ..modules import heuristics
 from ..modules.configs import (DSEmbeddingsConfig, DSLinearConfig, DSMoEConfig, DSNormConfig, DSRecurrentMixerConfig,
                                DSSelfAttentionConfig, DistanceBiasConfig, MaskingType, PositionalEmbeddingType,
@@ -47,7 +50,8 @@ from .inference_transformer_base import DSInferenceModelBase, LayerWeights
 
 @dataclass
 class HybridLayerSpec:
-    kind: str                      # "attention" | "latent_attention" | "delta" | "channel_delta" | "ssd" | "mlstm"
+    # "attention" | "rotary_attention" | "latent_attention" | "delta" | "channel_delta" | "removal_delta" | "ssd" | "mlstm" | "pair"
+    kind: str
     n_heads: int
     n_heads_kv: int                             # key/value heads (attention), key/query heads (delta), groups (ssd)
     key_dim: int                                # query/key head size, or state size per group (ssd)
@@ -98,6 +102,17 @@ class HybridLayerSpec:
     moe_scale: float = 1.0
     moe_identity: int = 0
     ff_limit: float = 0.0
+    # rotary attention (``rot_dims``, ``rot_base``, ``window``, ``out_gate``, ``gate_per_head`` above): pairing, one divisor for all
+    # frequencies, norm over whole q / k rows, values = projected keys, one added to the softmax denominator, a number per head
+    rot_interleaved: bool = False
+    rot_divisor: float = 1.0
+    qk_row_norm: bool = False
+    values_from_keys: bool = False
+    unit_sink: bool = False
+    head_scale: bool = False
+    decay_rate: float = 1.0                     # removal delta: decay = exp(-decay_rate * sigmoid(.))
+    # pair: two mixers that read the same input; the layer's mixer output is half the sum of their RMS-normed outputs
+    parts: Optional[Tuple["HybridLayerSpec", "HybridLayerSpec"]] = None
 
 
 @dataclass
@@ -113,14 +128,14 @@ class HybridSpec:
     loop_times: int = 1
     dtype: torch.dtype = torch.bfloat16
     max_seq_len: int = 1 << 20
-    block_form: str = "sandwich"                # "sandwich" | "post_scaled" | "pre_scaled"
+    block_form: str = "sandwich"                # "sandwich" | "post_scaled" | "pre_scaled" | "parallel"
     residual_mult: float = 1.0                  # pre_scaled: what every sublayer's output is multiplied by
     token_side_dim: int = 0                     # pre_scaled: channels per layer of the per-layer token input (0: none)
     layer_scale: bool = False                   # pre_scaled: every sublayer's output times a per-channel ``ls1`` / ``ls2``
     norm_weight_offset: float = 0.0             # pre_scaled: norm weights are ``offset + w`` (1: stored around zero)
     logit_scale: float = 1.0
     logit_softcap: float = 0.0                  # > 0: logits <- cap * tanh(logits / cap)
-    input_conv_taps: int = 0                    # post_scaled: taps of the filter in front of every sublayer
+    input_conv_taps: int = 0                    # taps of the filter in front of every sublayer (post_scaled) or mixer (parallel)
     depth_mix: bool = False                     # post_scaled: every layer hands on a mixture of all results so far
 
     def runs(self) -> List[Tuple[int, bool]]:
@@ -152,7 +167,10 @@ class DSHybridModel(DSInferenceModelBase):
     ``layer_scale``: ``ls1``, ``ls2``.  Channel delta rule: ``conv_w``, ``A_log``, ``dt_bias`` (fp32), ``w_a2``, ``w_g2``,
     ``norm``; latent attention ``q_norm``, ``w_uq`` (not with direct queries), ``kv_norm``, ``w_uk``, ``w_uv_t``; three-power
     feed-forward ``w_up``, ``b_up``, ``w_down``, ``b_down``, ``act_coef`` (fp32); group-limited experts ``moe_gate``,
-    ``moe_correction`` (fp32), ``moe_w1``, ``moe_w2``.  Two entries of ``layers`` may be one object (borrowed weights)."""
+    ``moe_correction`` (fp32), ``moe_w1``, ``moe_w2``.  Two entries of ``layers`` may be one object (borrowed weights).
+    Parallel stacks: ``norm1``, ``norm2``, ``filter1`` (``[taps, width]``); rotary attention ``q_norm`` / ``k_norm``,
+    ``q_head_scale`` (fp32); a pair has one ``w_in`` for both mixers and ``parts``, two :class:`LayerWeights` with the mixers'
+    tensors, ``wo`` and ``out_norm``; removal delta ``w0``, ``a_bias`` (fp32), ``w2`` (``[rank, heads * dim]``), ``norm``."""
 
     def __init__(self, spec: HybridSpec, weights: Dict, engine_config: RaggedInferenceEngineConfig, state_manager=None,
                  base_mp_group=None) -> None:
@@ -172,8 +190,9 @@ class DSHybridModel(DSInferenceModelBase):
             torch.backends.cudnn.allow_tf32 = False
         self._runs = spec.runs()
         # which cache / state entries every execution of a layer uses
-        self._cache_of_run: Dict[int, int] = {}
-        self._state_of_run: Dict[int, Tuple[int, ...]] = {}
+        # (the mixers of a pair: under (run, 0) and (run, 1))
+        self._cache_of_run: Dict = {}
+        self._state_of_run: Dict = {}
         self._conv_of_run: Dict[int, Tuple[int, int]] = {}
         self.layer_outputs = None        # set to a list: the stream every layer run hands on is appended (a copy)
         self._build_modules()
@@ -195,7 +214,7 @@ class DSHybridModel(DSInferenceModelBase):
             self.post_norm = heuristics.instantiate_scaled_post_norm(DSNormConfig(
                 max_tokens=mt, type=NormTypeEnum.RMSNorm, channels=s.model_dim, residual_dtype=DtypeEnum.fp32,
                 input_dtype=dt, output_dtype=dt, eps=s.norm_eps), ec)
-        elif s.block_form not in ("sandwich", "pre_scaled"):
+        elif s.block_form not in ("sandwich", "pre_scaled", "parallel"):
             raise ValueError(f"unknown block form {s.block_form!r}")
         self.mixers, self.moes = [], []
         for L in s.layers:
@@ -215,76 +234,99 @@ class DSHybridModel(DSInferenceModelBase):
                     score_correction=L.moe_correction, n_groups=L.moe_groups, keep_groups=L.moe_keep_groups,
                     score_scale=L.moe_scale, identity_experts=L.moe_identity, activation_limit=L.ff_limit), ec)
             self.moes.append(moe)
-            if L.kind == "latent_attention":
-                mod = heuristics.instantiate_attention(DSSelfAttentionConfig(
-                    max_tokens=mt, n_heads_q=L.n_heads, n_heads_kv=1, head_size=L.key_dim, v_head_size=L.value_dim,
-                    max_sequences=sm.max_ragged_sequence_count, scale_factor=L.attn_scale, input_dtype=dt,
-                    output_dtype=dt,
-                    masking_type=MaskingType.sliding_window if L.window > 0 else MaskingType.causal,
-                    masking_args={"size": L.window} if L.window > 0 else {},
-                    positional_embedding_type=(PositionalEmbeddingType.rotate_every_other if L.rot_dims > 0
-                                               else PositionalEmbeddingType.none),
-                    positional_embedding_config=RotateHalfConfig(theta_base=L.rot_base, rotate_dim=L.rot_dims),
-                    qk_norm_eps=s.norm_eps, sink=L.sink, kv_latent_dim=L.kv_rank, rope_head_dim=L.rot_dim,
-                    output_gate=L.out_gate, output_gate_per_head=L.gate_per_head, q_direct=L.q_direct,
-                    rotary_scaling=None if L.rot_scaling is None else RotaryScalingConfig(
-                        factor=L.rot_scaling[0], original=L.rot_scaling[1], fast=L.rot_scaling[2],
-                        slow=L.rot_scaling[3])), ec)
-            elif L.kind == "attention" and (L.conv_taps > 1 or L.qk_norm_weight or L.dist_rows > 0 or L.out_gate
-                                            or L.q_temp_coef != 0.0):
-                mask = (MaskingType.chunked if L.chunk_size > 0 else
-                        MaskingType.sliding_window if L.window > 0 else MaskingType.causal)
-                mod = heuristics.instantiate_attention(DSSelfAttentionConfig(
-                    max_tokens=mt, n_heads_q=L.n_heads, n_heads_kv=L.n_heads_kv, head_size=L.key_dim,
-                    v_head_size=L.value_dim, max_sequences=sm.max_ragged_sequence_count, scale_factor=L.attn_scale,
-                    input_dtype=dt, output_dtype=dt, masking_type=mask,
-                    masking_args={"size": L.chunk_size or L.window} if mask != MaskingType.causal else {},
-                    positional_embedding_type=(PositionalEmbeddingType.distance_bias if L.dist_rows > 0
-                                               else PositionalEmbeddingType.none),
-                    distance_bias=DistanceBiasConfig(rows=L.dist_rows, far=L.dist_far) if L.dist_rows > 0 else None,
-                    qk_norm_eps=s.norm_eps, qkv_conv_taps=L.conv_taps, qk_norm_weight=L.qk_norm_weight,
-                    q_temp_coef=L.q_temp_coef, q_temp_every=L.q_temp_every, output_gate=L.out_gate), ec)
-            elif L.kind == "attention":
-                mod = heuristics.instantiate_attention(DSSelfAttentionConfig(
-                    max_tokens=mt, n_heads_q=L.n_heads, n_heads_kv=L.n_heads_kv, head_size=L.key_dim,
-                    v_head_size=L.value_dim, max_sequences=sm.max_ragged_sequence_count, scale_factor=L.attn_scale,
-                    input_dtype=dt, output_dtype=dt,
-                    masking_type=MaskingType.chunked if L.chunk_size > 0 else MaskingType.causal,
-                    masking_args={"size": L.chunk_size} if L.chunk_size > 0 else {},
-                    positional_embedding_type=PositionalEmbeddingType.none, qk_unit_rms=L.qk_unit_rms,
-                    qk_norm_eps=s.norm_eps, sink=L.sink), ec)
-            else:
-                mod = heuristics.instantiate_recurrent_mixer(DSRecurrentMixerConfig(
-                    max_tokens=mt, kind=L.kind, model_dim=s.model_dim, n_heads=L.n_heads, n_heads_kv=L.n_heads_kv,
-                    key_dim=L.key_dim, value_dim=L.value_dim, conv_taps=L.conv_taps, norm_groups=L.norm_groups,
-                    gate_cap=L.gate_cap, eps=s.norm_eps, max_sequences=sm.max_ragged_sequence_count, input_dtype=dt, output_dtype=dt), ec)
-            self.mixers.append(mod)
-        n_cache = 0
+            self.mixers.append(tuple(self._build_mixer(part) for part in L.parts) if L.kind == "pair" else self._build_mixer(L))
         self._state_cfg = StatePoolConfig()
         shapes = []
         for r, (li, _) in enumerate(self._runs):
             L = s.layers[li]
-            if L.kind == "attention":
-                self._cache_of_run[r] = n_cache
-                shapes.append((L.n_heads_kv, L.key_dim, L.value_dim))
-                n_cache += 1
-                if hasattr(self.mixers[li], "state_shapes"):        # carried inputs of filtered projections
-                    self._state_of_run[r] = tuple(self._state_cfg.add(shape, sdt)
-                                                  for shape, sdt in self.mixers[li].state_shapes())
-            elif L.kind == "latent_attention":
-                self._cache_of_run[r] = n_cache
-                shapes.append((1, self.mixers[li].cache_row, 0))        # latent | rotated key part; no value tensor
-                n_cache += 1
+            if L.kind == "pair":
+                for j, part in enumerate(L.parts):
+                    self._plan_memory((r, j), part, self.mixers[li][j], shapes)
             else:
-                self._state_of_run[r] = tuple(self._state_cfg.add(shape, sdt)
-                                              for shape, sdt in self.mixers[li].state_shapes())
+                self._plan_memory(r, L, self.mixers[li], shapes)
             if s.block_form == "post_scaled":
                 # the last taps - 1 inputs of the filter in front of the mixer and of the one in front of the feed-forward
                 keep = (max(s.input_conv_taps, 1) - 1, s.model_dim)
                 self._conv_of_run[r] = (self._state_cfg.add(keep, torch.float32),
                                         self._state_cfg.add(keep, torch.float32) if L.ff_dim > 0 else -1)
+            elif s.block_form == "parallel":
+                keep = (max(s.input_conv_taps, 1) - 1, s.model_dim)
+                self._conv_of_run[r] = (self._state_cfg.add(keep, torch.float32) if keep[0] > 0 else -1, -1)
         self._cache_shapes = tuple(shapes)
         self._stack = None
+
+    def _build_mixer(self, L: HybridLayerSpec):
+        s, ec = self.spec, self._engine_config
+        sm = ec.state_manager
+        dt, mt = DtypeEnum(s.dtype), sm.max_ragged_batch_size
+        if L.kind == "latent_attention":
+            return heuristics.instantiate_attention(DSSelfAttentionConfig(
+                max_tokens=mt, n_heads_q=L.n_heads, n_heads_kv=1, head_size=L.key_dim, v_head_size=L.value_dim,
+                max_sequences=sm.max_ragged_sequence_count, scale_factor=L.attn_scale, input_dtype=dt,
+                output_dtype=dt,
+                masking_type=MaskingType.sliding_window if L.window > 0 else MaskingType.causal,
+                masking_args={"size": L.window} if L.window > 0 else {},
+                positional_embedding_type=(PositionalEmbeddingType.rotate_every_other if L.rot_dims > 0
+                                           else PositionalEmbeddingType.none),
+                positional_embedding_config=RotateHalfConfig(theta_base=L.rot_base, rotate_dim=L.rot_dims),
+                qk_norm_eps=s.norm_eps, sink=L.sink, kv_latent_dim=L.kv_rank, rope_head_dim=L.rot_dim,
+                output_gate=L.out_gate, output_gate_per_head=L.gate_per_head, q_direct=L.q_direct,
+                rotary_scaling=None if L.rot_scaling is None else RotaryScalingConfig(
+                    factor=L.rot_scaling[0], original=L.rot_scaling[1], fast=L.rot_scaling[2],
+                    slow=L.rot_scaling[3])), ec)
+        if L.kind == "attention" and (L.conv_taps > 1 or L.qk_norm_weight or L.dist_rows > 0 or L.out_gate
+                                        or L.q_temp_coef != 0.0):
+            mask = (MaskingType.chunked if L.chunk_size > 0 else
+                    MaskingType.sliding_window if L.window > 0 else MaskingType.causal)
+            return heuristics.instantiate_attention(DSSelfAttentionConfig(
+                max_tokens=mt, n_heads_q=L.n_heads, n_heads_kv=L.n_heads_kv, head_size=L.key_dim,
+                v_head_size=L.value_dim, max_sequences=sm.max_ragged_sequence_count, scale_factor=L.attn_scale,
+                input_dtype=dt, output_dtype=dt, masking_type=mask,
+                masking_args={"size": L.chunk_size or L.window} if mask != MaskingType.causal else {},
+                positional_embedding_type=(PositionalEmbeddingType.distance_bias if L.dist_rows > 0
+                                           else PositionalEmbeddingType.none),
+                distance_bias=DistanceBiasConfig(rows=L.dist_rows, far=L.dist_far) if L.dist_rows > 0 else None,
+                qk_norm_eps=s.norm_eps, qkv_conv_taps=L.conv_taps, qk_norm_weight=L.qk_norm_weight,
+                q_temp_coef=L.q_temp_coef, q_temp_every=L.q_temp_every, output_gate=L.out_gate), ec)
+        if L.kind == "attention":
+            return heuristics.instantiate_attention(DSSelfAttentionConfig(
+                max_tokens=mt, n_heads_q=L.n_heads, n_heads_kv=L.n_heads_kv, head_size=L.key_dim,
+                v_head_size=L.value_dim, max_sequences=sm.max_ragged_sequence_count, scale_factor=L.attn_scale,
+                input_dtype=dt, output_dtype=dt,
+                masking_type=MaskingType.chunked if L.chunk_size > 0 else MaskingType.causal,
+                masking_args={"size": L.chunk_size} if L.chunk_size > 0 else {},
+                positional_embedding_type=PositionalEmbeddingType.none, qk_unit_rms=L.qk_unit_rms,
+                qk_norm_eps=s.norm_eps, sink=L.sink), ec)
+        if L.kind == "rotary_attention":
+            return heuristics.instantiate_attention(DSSelfAttentionConfig(
+                max_tokens=mt, n_heads_q=L.n_heads, n_heads_kv=L.n_heads_kv, head_size=L.key_dim, v_head_size=L.value_dim,
+                max_sequences=sm.max_ragged_sequence_count, scale_factor=L.attn_scale, input_dtype=dt, output_dtype=dt,
+                masking_type=MaskingType.sliding_window if L.window > 0 else MaskingType.causal,
+                masking_args={"size": L.window} if L.window > 0 else {},
+                positional_embedding_type=(PositionalEmbeddingType.none if L.rot_dims == 0 else
+                                           PositionalEmbeddingType.rotate_every_other if L.rot_interleaved else
+                                           PositionalEmbeddingType.rotate_half),
+                positional_embedding_config=RotateHalfConfig(theta_base=L.rot_base, rotate_dim=L.rot_dims,
+                                                             freq_divisor=L.rot_divisor),
+                qk_norm_eps=s.norm_eps, split_cache=True, qk_row_norm=L.qk_row_norm, values_from_keys=L.values_from_keys,
+                unit_sink=L.unit_sink, sink=L.sink, q_head_scale=L.head_scale, output_gate=L.out_gate,
+                output_gate_per_head=L.gate_per_head), ec)
+        return heuristics.instantiate_recurrent_mixer(DSRecurrentMixerConfig(
+            max_tokens=mt, kind=L.kind, model_dim=s.model_dim, n_heads=L.n_heads, n_heads_kv=L.n_heads_kv,
+            key_dim=L.key_dim, value_dim=L.value_dim, conv_taps=L.conv_taps, norm_groups=L.norm_groups,
+            gate_cap=L.gate_cap, decay_rate=L.decay_rate, eps=s.norm_eps, max_sequences=sm.max_ragged_sequence_count,
+            input_dtype=dt, output_dtype=dt), ec)
+
+    def _plan_memory(self, key, L: HybridLayerSpec, mod, shapes: List) -> None:
+        """Cache and state entries of one execution of a mixer (``key``: the run, or (run, part) in a pair)."""
+        if L.kind in ("attention", "rotary_attention"):
+            self._cache_of_run[key] = len(shapes)
+            shapes.append((L.n_heads_kv, L.key_dim, L.value_dim))
+        elif L.kind == "latent_attention":
+            self._cache_of_run[key] = len(shapes)
+            shapes.append((1, mod.cache_row, 0))        # latent | rotated key part; no value tensor
+        if hasattr(mod, "state_shapes"):                # recurrences; carried inputs of filtered projections
+            self._state_of_run[key] = tuple(self._state_cfg.add(shape, sdt) for shape, sdt in mod.state_shapes())
 
     # ------------------------------------------------------------------------------------------ properties
     @property
@@ -351,20 +393,31 @@ class DSHybridModel(DSInferenceModelBase):
             h = M.gated_act_rows(h, L.ff_activation)
         return self.linear(h, lw.w_down)
 
-    def _mixer(self, r: int, li: int, lw: LayerWeights, x: torch.Tensor, batch) -> torch.Tensor:
-        L, mod, sm = self.spec.layers[li], self.mixers[li], self.state_manager
-        proj = self.linear(x, lw.w_in)
+    def _mix(self, key, L: HybridLayerSpec, mod, lw: LayerWeights, proj: torch.Tensor, batch) -> torch.Tensor:
+        """A mixer on its projection columns, before its output projection."""
+        sm = self.state_manager
         if L.kind == "attention" and hasattr(mod, "filtered_channels"):
-            states = self._state_of_run.get(r, ())
-            ctx = mod(proj, sm.get_cache(self._cache_of_run[r]), batch, None, lw,
-                      sm.get_state(states[0]) if states else None)
-        elif L.kind == "attention":
-            ctx = mod(proj, sm.get_cache(self._cache_of_run[r]), batch, None, lw.b_in, lw.sink)
-        elif L.kind == "latent_attention":
-            ctx = mod(proj, sm.get_cache(self._cache_of_run[r]), batch, None, lw)
-        else:
-            ctx = mod(proj, lw, tuple(sm.get_state(e) for e in self._state_of_run[r]), batch)
+            states = self._state_of_run.get(key, ())
+            return mod(proj, sm.get_cache(self._cache_of_run[key]), batch, None, lw,
+                       sm.get_state(states[0]) if states else None)
+        if L.kind == "attention":
+            return mod(proj, sm.get_cache(self._cache_of_run[key]), batch, None, lw.b_in, lw.sink)
+        if L.kind in ("latent_attention", "rotary_attention"):
+            return mod(proj, sm.get_cache(self._cache_of_run[key]), batch, None, lw)
+        return mod(proj, lw, tuple(sm.get_state(e) for e in self._state_of_run[key]), batch)
+
+    def _mixer(self, r: int, li: int, lw: LayerWeights, x: torch.Tensor, batch) -> torch.Tensor:
+        ctx = self._mix(r, self.spec.layers[li], self.mixers[li], lw, self.linear(x, lw.w_in), batch)
         return self.linear(ctx, lw.wo)
+
+    def _mixer_pair(self, r: int, li: int, lw: LayerWeights, x: torch.Tensor, batch) -> P.StreamSum:
+        """Both mixers of a pair on one fused projection; their norms and average happen where the sum joins the stream."""
+        L, mods = self.spec.layers[li], self.mixers[li]
+        proj = self.linear(x, lw.w_in)
+        cut = mods[0].projection_width
+        a, b = (self.linear(self._mix((r, j), L.parts[j], mods[j], lw.parts[j], cols, batch), lw.parts[j].wo)
+                for j, cols in enumerate((proj[:, :cut], proj[:, cut:])))
+        return P.StreamSum(a=a, wa=lw.parts[0].out_norm, b=b, wb=lw.parts[1].out_norm, mult=0.5)
 
     def _filtered(self, x: torch.Tensor, w: torch.Tensor, entry: int, batch) -> torch.Tensor:
         """What a sublayer of a post-scaled layer reads: ``x + filter(x)`` in the activation dtype; the sequence's
@@ -460,8 +513,40 @@ class DSHybridModel(DSInferenceModelBase):
         return logits
 
     @torch.no_grad()
+    def _forward_parallel(self, batch) -> torch.Tensor:
+        """Layers ``x <- x + mixer(c(norm1(x))) + ff(norm2(x))``.  What a layer adds stays pending (``add``) until the kernel that
+        adds it also computes both inputs of the next layer (one kernel in a decode step, two for prompt rows)."""
+        W, s = self.weights, self.spec
+        info, t2s, single = batch.seq_info(), batch.token_to_seq(), batch.single_rows()
+        resid = self.embed(batch, W["embed"])
+        add = None
+        for r, (li, _) in enumerate(self._runs):
+            lw, L = W["layers"][li], s.layers[li]
+            entry = self._conv_of_run[r][0]
+            x, xf = P.open_parallel_layer(resid, add, lw.norm1, lw.filter1,
+                                          self.state_manager.get_state(entry) if entry >= 0 else None,
+                                          lw.norm2 if L.ff_dim > 0 else None, s.norm_eps, s.dtype, info, t2s, single)
+            if L.kind == "pair":
+                add = self._mixer_pair(r, li, lw, x, batch)
+            else:
+                add = P.StreamSum(a=self._mixer(r, li, lw, x, batch))
+            if L.ff_dim > 0:
+                add.y = self._feed_forward(L, lw, xf, li)
+            if self.layer_outputs is not None:
+                P.stream_add(resid, add, s.norm_eps, s.dtype)
+                add = None
+                self.layer_outputs.append(resid.clone())
+        rows = batch.last_token_index()
+        if rows.numel() == 0:               # a step that only advances caches and states
+            return torch.empty(0, s.vocab_size, dtype=torch.float32, device=resid.device)
+        h = P.stream_norm_rows(resid, add, rows, W["final_norm_w"], s.norm_eps, s.dtype)
+        return self.linear(h, W["unembed"])[:, : s.vocab_size].float()
+
+    @torch.no_grad()
     def forward(self, batch) -> torch.Tensor:
         W, s = self.weights, self.spec
+        if s.block_form == "parallel":
+            return self._forward_parallel(batch)
         if s.block_form == "post_scaled":
             return self._forward_post_scaled(batch)
         if s.block_form == "pre_scaled":

@@ -276,8 +276,9 @@ from .fomalix import FomalixPolicy  # noqa: E402
 from .kekopel import KekopelPolicy  # noqa: E402
 from .ridazen import RidazenPolicy  # noqa: E402
 from .pifazen import PifazenPolicy  # noqa: E402
+from .vezodra import VezodraPolicy  # noqa: E402
 
-POLICIES = {"fomalix": FomalixPolicy, "kekopel": KekopelPolicy, "ridazen": RidazenPolicy, "pifazen": PifazenPolicy,
+POLICIES = {"fomalix": FomalixPolicy, "kekopel": KekopelPolicy, "ridazen": RidazenPolicy, "pifazen": PifazenPolicy, "vezodra": VezodraPolicy,
             "llama": Llama2Policy, "mistral": MistralPolicy, "mixtral": MixtralPolicy, "falcon": FalconPolicy,
             "opt": OPTPolicy, "phi": PhiPolicy, "phi3": Phi3Policy, "qwen": QwenPolicy, "qwen2": Qwen2Policy,
             "qwen2_moe": Qwen2MoePolicy}

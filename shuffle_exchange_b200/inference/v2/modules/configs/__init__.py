@@ -26,6 +26,7 @@ class RotateHalfConfig(DeepSpeedConfigModel):
     use_trained_freqs: bool = False
     theta_base: float = 10_000.0
     rotate_dim: Optional[int] = None      # None: rotate the whole head; < head_size: partial rotary (Phi, GPT-NeoX)
+    freq_divisor: float = 1.0             # linear scaling: every angular frequency is divided by this
 
 
 class RotaryScalingConfig(DeepSpeedConfigModel):
@@ -85,6 +86,12 @@ class DSSelfAttentionConfig(DSModuleConfig):
     # at the start of the fused projection) instead of through a normalised latent with an up-projection.
     q_direct: bool = False
     rotary_scaling: Optional[RotaryScalingConfig] = None
+    # Rotated attention whose keys and values live in two paged tensors (their head sizes may differ).
+    split_cache: bool = False
+    qk_row_norm: bool = False             # RMS norm over ALL query (key) heads of a token at once, one weight per channel
+    values_from_keys: bool = False        # the values are the projected keys before rotation (no value projection)
+    unit_sink: bool = False               # one is added to the softmax denominator (a sink logit of zero on every head)
+    q_head_scale: bool = False            # the scores of every query head are multiplied by a learned number
 
 
 class DSEmbeddingsConfig(DSModuleConfig):
@@ -162,7 +169,9 @@ class DSRecurrentMixerConfig(DSModuleConfig):
     projection behind the per-head norm.  ``"ssd"``: state-space duality (B / C of ``key_dim`` = state size per
     group, a convolution over x | B | C, a skip term and a gated group norm).  ``"mlstm"``: matrix-memory LSTM
     (exponential input gate, sigmoid forget gate in log space, both capped by ``gate_cap``, a running maximum that
-    keeps the exponentials in range, a normaliser state, per-head unit-RMS and a sigmoid output gate; no convolution)."""
+    keeps the exponentials in range, a normaliser state, per-head unit-RMS and a sigmoid output gate; no convolution).
+    ``"removal_delta"``: a delta rule whose decay, and whose rate of removing what a key has stored, are vectors over the key
+    channels of every head (no convolution, key and value sizes equal; ``decay_rate`` bounds the decay from below)."""
     kind: str
     model_dim: int
     n_heads: int
@@ -172,6 +181,7 @@ class DSRecurrentMixerConfig(DSModuleConfig):
     conv_taps: int = 1
     norm_groups: int = 1
     gate_cap: float = 0.0                 # mlstm: gate pre-activations pass cap * tanh(x / cap)
+    decay_rate: float = 1.0               # removal_delta: decay = exp(-decay_rate * sigmoid(.))
     eps: float = 1e-5
     unit_norm_eps: float = 1e-6
     max_sequences: int = 1

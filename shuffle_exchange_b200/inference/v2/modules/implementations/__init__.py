@@ -23,6 +23,9 @@
                               state per (sequence slot, head) + gated group norm
  ``channel_delta_mixer``      the delta rule with a separate decay for every key channel of every head and a sigmoid output gate, both
                               from two-step projections
+ ``rotary_sink_attention``    rotation in either pairing, whole-row q/k norm, values that may be the unrotated keys, causal or
+                              windowed softmax that may add one to its denominator, a scale and an output gate per head
+ ``removal_delta_mixer``      delta rule with a decay and a removal rate per head and key channel
 =========================  =======================================================================================
 """
 from __future__ import annotations
@@ -38,6 +41,7 @@ from ...inference_parameter import InferenceParameter
 from ...inference_utils import ActivationType, DtypeEnum, NormTypeEnum, is_gated
 from ...kernels import ragged_ops as R
 from ...kernels import mixer_ops as M
+from ...kernels import parallel_ops as P
 from ..configs import (DSEmbeddingsConfig, DSLinearConfig, DSMoEConfig, DSNormConfig, DSRecurrentMixerConfig,
                        DSSelfAttentionConfig, DSUnembedConfig, MaskingType, PositionalEmbeddingType)
 from ..interfaces import (DSEmbeddingBase, DSEmbeddingRegistry, DSLinearBase, DSLinearRegistry, DSMoEBase,
@@ -86,7 +90,7 @@ class DSDenseBlockedAttention(DSSelfAttentionBase):
 
     @staticmethod
     def supports_config(config: DSSelfAttentionConfig) -> bool:
-        if MaskingType(config.masking_type) != MaskingType.causal:
+        if MaskingType(config.masking_type) != MaskingType.causal or config.split_cache:
             return False
         if config.sink or config.qk_unit_rms or config.v_head_size not in (None, config.head_size):
             return False
@@ -433,6 +437,9 @@ class DSSinkChunkedAttention(DSSelfAttentionBase):
         if MaskingType(config.masking_type) == MaskingType.chunked and int(config.masking_args.get("size", 0)) < 1:
             return False
         if config.qkv_conv_taps > 1 or config.qk_norm_weight or config.q_temp_coef != 0.0 or config.output_gate:
+            return False
+        if (config.split_cache or config.qk_row_norm or config.values_from_keys or config.unit_sink
+                or config.q_head_scale):
             return False
         return (PositionalEmbeddingType(config.positional_embedding_type) == PositionalEmbeddingType.none
                 and (config.v_head_size or config.head_size) <= 256 and config.n_heads_q % config.n_heads_kv == 0)
@@ -884,6 +891,9 @@ class DSFilteredBiasAttention(DSSelfAttentionBase):
     def supports_config(config: DSSelfAttentionConfig) -> bool:
         if config.kv_latent_dim is not None or config.sink:
             return False
+        if (config.split_cache or config.qk_row_norm or config.values_from_keys or config.unit_sink
+                or config.q_head_scale or config.output_gate_per_head):
+            return False
         if MaskingType(config.masking_type) not in (MaskingType.causal, MaskingType.chunked, MaskingType.sliding_window):
             return False
         pe = PositionalEmbeddingType(config.positional_embedding_type)
@@ -963,3 +973,149 @@ class DSFilteredBiasAttention(DSSelfAttentionBase):
         gate = projected[:, C: C + c.n_heads_q * dv] if c.output_gate else None
         return M.sink_attention(q, keys, values, None, t2s, pos, tables, c.scale_factor, chunk, _dt(c.output_dtype).torch,
                                 atoms, n_long, window=window, dist_bias=bias, gate=gate)
+
+
+@DSSelfAttentionRegistry.register_module
+class DSRotarySinkAttention(DSSelfAttentionBase):
+    """Softmax attention with rotated queries and keys over a pair of paged caches.  Projection columns: ``q (Hq d) | k (G d) | v
+    (G dv) | gate``, without the v columns when the values are the projected keys themselves (``values_from_keys``: as projected,
+    before rotation), the gate (one column per head, or per output channel) starting at the next multiple of 8.  Optional RMS
+    norm over the whole q (k) row with a weight per channel (``qk_row_norm``), rotation of the first channels of every head in
+    either pairing with all frequencies divided by one factor, a learned number per query head on the scores, causal /
+    chunk-local / sliding-window mask, one added to the softmax denominator (``unit_sink``) or a learned sink logit.  Norms,
+    angles, scores, weights and the weighted sum are fp32.
+
+    ``forward(projected, (keys, values), batch, inv_freqs, weights)``: ``weights`` has ``q_norm`` / ``k_norm``, ``q_head_scale``
+    (fp32 ``[Hq]``) and ``sink`` (fp32 ``[Hq]``) as far as the configuration asks for them."""
+
+    @staticmethod
+    def name() -> str:
+        return "rotary_sink_attention"
+
+    @staticmethod
+    def supports_config(config: DSSelfAttentionConfig) -> bool:
+        if config.kv_latent_dim is not None or config.qkv_conv_taps > 1 or config.q_temp_coef != 0.0:
+            return False
+        if config.qk_unit_rms or config.qk_norm_weight or config.rotary_scaling is not None or (config.sink and config.unit_sink):
+            return False
+        if MaskingType(config.masking_type) not in (MaskingType.causal, MaskingType.chunked, MaskingType.sliding_window):
+            return False
+        if MaskingType(config.masking_type) != MaskingType.causal and int(config.masking_args.get("size", 0)) < 1:
+            return False
+        dv = config.v_head_size or config.head_size
+        if config.values_from_keys and dv != config.head_size:
+            return False
+        return (PositionalEmbeddingType(config.positional_embedding_type) in (
+            PositionalEmbeddingType.none, PositionalEmbeddingType.rotate_half, PositionalEmbeddingType.rotate_every_other)
+            and config.head_size <= 256 and dv <= 256 and config.n_heads_q % config.n_heads_kv == 0)
+
+    def __init__(self, config: DSSelfAttentionConfig, implementation_config: Dict[str, Any]) -> None:
+        super().__init__(config, implementation_config)
+        pe, rot = PositionalEmbeddingType(config.positional_embedding_type), config.positional_embedding_config
+        n_rot = 0
+        if pe != PositionalEmbeddingType.none:
+            n_rot = config.head_size if rot is None or rot.rotate_dim is None else rot.rotate_dim
+        if n_rot % 2 or n_rot > config.head_size:
+            raise ValueError(f"cannot rotate {n_rot} of {config.head_size} channels in pairs")
+        self._interleaved = pe == PositionalEmbeddingType.rotate_every_other
+        self._inv_freq = self.rotary_table(n_rot, 10000.0 if rot is None else rot.theta_base,
+                                           1.0 if rot is None else rot.freq_divisor)
+        self._zero_sink = torch.zeros(config.n_heads_q, dtype=torch.float32) if config.unit_sink else None
+
+    @staticmethod
+    def rotary_table(n_rot: int, base: float, divisor: float = 1.0) -> torch.Tensor:
+        """fp32 angular frequencies ``base^(-2i / n_rot) / divisor`` of the ``n_rot / 2`` pairs, evaluated in float64."""
+        i = torch.arange(0, n_rot, 2, dtype=torch.float64)
+        return (torch.pow(torch.tensor(float(base), dtype=torch.float64), -i / max(n_rot, 1)) / divisor).to(torch.float32)
+
+    @property
+    def kv_block_size(self) -> int:
+        return 64
+
+    @property
+    def q_block_size(self) -> int:
+        return 1
+
+    @property
+    def projection_width(self) -> int:
+        """Columns of the projection block, its padding to whole 16-byte words included."""
+        c, g = self._config, 0
+        if c.output_gate:
+            g = c.n_heads_q * (1 if c.output_gate_per_head else (c.v_head_size or c.head_size))
+        return self.gate_column + (g + 7) // 8 * 8
+
+    @property
+    def gate_column(self) -> int:
+        c = self._config
+        n = (c.n_heads_q + c.n_heads_kv) * c.head_size
+        if not c.values_from_keys:
+            n += c.n_heads_kv * (c.v_head_size or c.head_size)
+        return (n + 7) // 8 * 8
+
+    def forward(self, projected: torch.Tensor, kv_cache, batch, inv_freqs=None, weights=None) -> torch.Tensor:
+        c = self._config
+        H, G, d, dv = c.n_heads_q, c.n_heads_kv, c.head_size, c.v_head_size or c.head_size
+        keys, values = kv_cache
+        if self._inv_freq.device != projected.device:
+            self._inv_freq = self._inv_freq.to(projected.device)
+            if self._zero_sink is not None:
+                self._zero_sink = self._zero_sink.to(projected.device)
+        t2s, pos, tables = batch.token_to_seq(), batch.token_positions(), batch.block_tables()
+        k0 = H * d
+        q = P.rope_append(projected, 0, k0, k0 if c.values_from_keys else k0 + G * d,
+                          weights.q_norm if c.qk_row_norm else None, weights.k_norm if c.qk_row_norm else None,
+                          self._inv_freq, self._interleaved, weights.q_head_scale if c.q_head_scale else None, keys, values,
+                          t2s, pos, tables, H, G, d, dv, c.qk_norm_eps)
+        mt = MaskingType(c.masking_type)
+        chunk = int(c.masking_args["size"]) if mt == MaskingType.chunked else 0
+        window = int(c.masking_args["size"]) if mt == MaskingType.sliding_window else 0
+        gate = None
+        if c.output_gate:
+            gate = projected[:, self.gate_column: self.gate_column + (H if c.output_gate_per_head else H * dv)]
+        atoms, n_long = None, 0
+        if q.is_cuda and M.tiles_supported(d, dv) and hasattr(batch, "atoms_longer_than"):
+            atoms, n_long = batch.atoms(), batch.atoms_longer_than(M.SHORT_ATOM)
+        sink = self._zero_sink if c.unit_sink else (weights.sink if c.sink else None)
+        return M.sink_attention(q, keys, values, sink, t2s, pos, tables, c.scale_factor, chunk, _dt(c.output_dtype).torch,
+                                atoms, n_long, window=window, gate=gate)
+
+
+@DSRecurrentMixerRegistry.register_module
+class DSRemovalDeltaMixer(_RecurrentMixer):
+    """Delta rule that removes and forgets at separate rates.  Projection columns (blocks padded to multiples of 8): ``r | k | v |
+    a | g (H n each) | low (rank)``.  Per head, with ``u = k / sqrt(sum k^2 + unit_norm_eps)``: decay ``w = exp(-decay_rate *
+    sigmoid(tanh(low) w2 + w0))`` and removal rate ``a = sigmoid(a + a_bias)`` per key channel, ``S <- diag(w) S - (a u) (u^T S) +
+    k v^T`` (both products read the old state), ``o = S^T r``; the output is ``o / rms(o) * norm * sigmoid(g)`` with ``rms`` per
+    head.  ``weights``: ``w2`` ``[rank, H n]``, ``w0`` and ``a_bias`` fp32 ``[H n]``, ``norm`` ``[H n]``."""
+
+    @staticmethod
+    def name() -> str:
+        return "removal_delta_mixer"
+
+    @staticmethod
+    def supports_config(config: DSRecurrentMixerConfig) -> bool:
+        return (config.kind == "removal_delta" and config.key_dim <= 256 and config.key_dim == config.value_dim
+                and config.n_heads == config.n_heads_kv and config.conv_taps <= 1 and config.decay_rate > 0.0)
+
+    @property
+    def conv_channels(self) -> int:
+        return 0
+
+    @property
+    def block_width(self) -> int:
+        """Columns of each of the five ``H n`` blocks, padding included."""
+        return (self._config.n_heads * self._config.key_dim + 7) // 8 * 8
+
+    def state_shapes(self):
+        c = self._config
+        return [((c.n_heads, c.value_dim, c.key_dim), torch.float32)]
+
+    def forward(self, projected, weights, states, batch):
+        c = self._config
+        H, n, B = c.n_heads, c.key_dim, self.block_width
+        (S,) = states
+        buf = P.removal_prepare(projected, 0, B, 2 * B, 3 * B, 5 * B, weights.w2, weights.w0, weights.a_bias, H, n,
+                                c.decay_rate, c.unit_norm_eps)
+        o = P.removal_recurrence(buf, S, batch.seq_info(), batch.single_rows())
+        return M.group_norm_gate(o, projected[:, 4 * B: 4 * B + H * n], weights.norm, n, c.eps, False,
+                                 _dt(c.output_dtype).torch, sigmoid=True)

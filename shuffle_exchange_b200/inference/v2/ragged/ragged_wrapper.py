@@ -116,6 +116,10 @@ class RaggedBatchWrapper:
         """How many (leading) atoms have more than ``q_len`` queries; host-side, no synchronisation."""
         return int((self._atom_q_lens > q_len).sum()) if self._n_atoms else 0
 
+    def single_rows(self) -> bool:
+        """Whether every sequence of the batch brings exactly one token (a pure decode step); host-side."""
+        return self._n_tokens == self._n_seqs
+
     @property
     def current_tokens(self) -> int:
         return self._n_tokens
