@@ -15,7 +15,7 @@ from ....native import lib as _lib
 from .mixer_ops import _rms, _rows
 
 _lib.register({
-    "sxb_resid_sum_step": "pppppp" "ff" "pppppppppppp" "iii" "i" "p",
+    "sxb_resid_sum_step": "pppppp" "ff" "pppppppppp" "iii" "i" "p",
     "sxb_norm_filter_rows": "pppppppppp" "iiii" "i" "p",
     "sxb_rope_append": "p" "l" "iii" "pppppppppp" "iiiiiiiii" "f" "i" "p",
     "sxb_removal_prepare": "p" "l" "iiiii" "pppp" "iiii" "ff" "i" "p",

@@ -6,13 +6,17 @@ per-sequence info]`` and
 is uploaded with a single ``cudaMemcpyAsync`` in ``finalize`` (the reference uses three pinned "fast host buffers",
 ``ragged/csrc/fast_host_buffer.cu``).  The attention atoms (one per 128-query tile of a sequence, with the KV extent
 it attends to) are cut by the native scheduler ``sxbh_build_atoms`` (``csrc/host/ragged_host.cpp``) at ``finalize``
-and consumed by the tensor-core paged attention kernel (``sxb_attn_fwd_atoms``)."""
+and consumed by the tensor-core paged attention kernel (``sxb_attn_fwd_atoms``).
+
+The upload is asynchronous and forwards may be queued without a synchronisation between them, so the batches take turns over
+``STAGING_BUFFERS`` pinned buffers; a buffer is written again only when the upload that read it has completed."""
 from __future__ import annotations
 
 import torch
 
 ATOM_Q_BLOCK = 128          # query rows of one attention atom = the kernel's q tile
 ATOM_KV_BLOCK = 64
+STAGING_BUFFERS = 4
 
 
 class RaggedBatchWrapper:
@@ -24,7 +28,10 @@ class RaggedBatchWrapper:
         n = 4 * self.max_tokens + self.max_seqs * self.max_blocks + 6 * self.max_atoms + 4 * self.max_seqs
         self._seq_meta = torch.zeros(3, self.max_seqs, dtype=torch.int32)      # start / in-flight tokens / seen tokens
         pin = torch.cuda.is_available()
-        self._host = torch.zeros(n, dtype=torch.int32, pin_memory=pin)
+        self._staging = [torch.zeros(n, dtype=torch.int32, pin_memory=pin) for _ in range(STAGING_BUFFERS if pin else 1)]
+        self._uploaded = [None] * len(self._staging)          # per buffer: event behind the last upload from it
+        self._turn = 0
+        self._host = self._staging[0]
         self._dev = torch.zeros(n, dtype=torch.int32, device=self.device)
         self.clear()
 
@@ -34,6 +41,12 @@ class RaggedBatchWrapper:
         self._n_atoms = 0
         self._n_logit_rows = 0
         self._finalized = False
+        if self._uploaded[self._turn] is not None:            # the current buffer is in use by an upload: take the next one
+            self._turn = (self._turn + 1) % len(self._staging)
+            if self._uploaded[self._turn] is not None:
+                self._uploaded[self._turn].synchronize()
+                self._uploaded[self._turn] = None
+            self._host = self._staging[self._turn]
 
     def _views(self, buf):
         T, S, B = self.max_tokens, self.max_seqs, self.max_blocks
@@ -82,6 +95,9 @@ class RaggedBatchWrapper:
             live.copy_(live[order])
             self._atom_q_lens = live[:, 2].clone()
         self._dev.copy_(self._host, non_blocking=True)
+        if self._dev.is_cuda:
+            ev = self._uploaded[self._turn] = torch.cuda.Event()
+            ev.record()
         self._finalized = True
 
     # device views ------------------------------------------------------------------------------
