@@ -8,7 +8,9 @@ Ridazen stack (attention with filtered projections, distance-bucket bias and out
 shared expert, per-layer token input) next to a Fomalix stack of attention layers only at equal size.  With
 ``--serve-model pifazen`` the pair is a Pifazen stack (latent attention with output gates and scaled rotation, a delta rule
 with a decay per key channel, three-power dense feed-forward, clamped experts chosen among groups with identity experts)
-next to the Kekopel stack of equal size whose window holds every key.
+next to the Kekopel stack of equal size whose window holds every key.  With ``--serve-model vezodra`` the pair is a Vezodra
+stack (mixer and feed-forward of one stream, rotary attention, windowed attention beside a delta rule with removal and decay
+vectors) next to a Fomalix stack of attention and delta-rule layers of equal size.
 
 Timing: CUDA events on the launching stream, >= 3 warm-up forwards, a buffer larger than L2 is rewritten between timed
 forwards.  Prefill: one request of ``prefill`` tokens in one forward.  Decode: ``batch`` requests with ``context`` tokens
@@ -940,6 +942,192 @@ def pifazen_kernel_table(z: Dict, prefill: int, batch: int, context: int, timer,
     return rows
 
 
+# ------------------------------------------------------------------------------------------------ Vezodra beside Fomalix
+VEZODRA = dict(taps=4, rank=64)
+
+
+def vezodra_config(z: Dict) -> Dict:
+    """Layers cycle attention / pair / pair; the window of the pairs' attention is :data:`WINDOW`."""
+    d, H, G = z["head"], z["heads"], z["kv_heads"]
+    att = {"dim": d, "heads": H, "kv_heads": G, "rot": {"base": 10000.0, "dims": d}, "scale": d ** -0.5, "vdim": d}
+    left = dict(att, mask={"size": WINDOW}, rot={"base": 10000.0, "dims": d, "scaling": {"factor": 4.0}})
+    kinds = [("attention", att)] + [("parallel", {"left": left, "right": {"dim": d, "heads": H}})] * 2
+    layers = [{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1], "mlp": {"ff": z["ff"], "kind": "dense"}}
+              for i in range(z["layers"])]
+    return {"architecture": "Vezodra", "canon": {"taps": VEZODRA["taps"]}, "layers": layers, "norm": {"eps": 1e-5},
+            "vocab": VOCAB, "width": z["width"]}
+
+
+def vezodra_weights(cfg: Dict, device) -> Dict[str, torch.Tensor]:
+    g = torch.Generator(device=device).manual_seed(0)
+    W, bf, rk = cfg["width"], torch.bfloat16, VEZODRA["rank"]
+
+    def mat(o, i):
+        return (torch.randn(o, i, generator=g, device=device) / math.sqrt(i)).to(bf)
+
+    def vec(n, lo=0.5, hi=1.5):
+        return (torch.rand(n, generator=g, device=device) * (hi - lo) + lo).to(bf)
+
+    out = {"embed": mat(cfg["vocab"], W), "final.norm": vec(W)}
+    for i, L in enumerate(cfg["layers"]):
+        m, p = L["mixer"], f"l{i}."
+        out[p + "norm1"], out[p + "norm2"] = vec(W), vec(W)
+        out[p + "canon1"] = vec(W * VEZODRA["taps"], -0.3, 0.3).view(W, VEZODRA["taps"])
+        if L["type"] == "attention":
+            H, G, d = m["heads"], m["kv_heads"], m["dim"]
+            out[p + "mix.q"], out[p + "mix.k"], out[p + "mix.g"] = mat(H * d, W), mat(G * d, W), mat(H, W)
+            out[p + "mix.temp"], out[p + "mix.o"] = vec(H), mat(W, H * d)
+        else:
+            a, b, q = m["left"], m["right"], p + "mix.left."
+            H, G, d, dv = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            out[q + "q"], out[q + "k"], out[q + "v"] = mat(H * d, W), mat(G * d, W), mat(G * dv, W)
+            out[q + "q.norm"], out[q + "k.norm"], out[q + "o"], out[q + "out"] = vec(H * d), vec(G * d), mat(W, H * dv), vec(W)
+            n, q = b["heads"] * b["dim"], p + "mix.right."
+            for name in ("r", "k", "v", "g", "a"):
+                out[q + name] = mat(n, W)
+            out[q + "a.b"], out[q + "w0"], out[q + "w1"], out[q + "w2"] = vec(n, -1, 1), vec(n, -3, 1), mat(rk, W), mat(n, rk)
+            out[q + "norm"], out[q + "o"], out[q + "out"] = vec(n), mat(W, n), vec(W)
+        ff = L["mlp"]["ff"]
+        out[p + "mlp.gate"], out[p + "mlp.up"], out[p + "mlp.down"] = mat(ff, W), mat(ff, W), mat(W, ff)
+    return out
+
+
+def build_vezodra(z: Dict, max_tokens: int, max_seqs: int, pages: int):
+    cfg = vezodra_config(z)
+    return build_engine_from_state_dict(cfg, vezodra_weights(cfg, "cuda"), _engine_config(max_tokens, max_seqs, pages),
+                                        dtype=torch.bfloat16)
+
+
+def build_attention_delta_stack(z: Dict, max_tokens: int, max_seqs: int, pages: int):
+    """The Fomalix stack with attention and delta-rule layers in turn (attention / delta / attention)."""
+    cfg = hybrid_config(z, kinds=("attention", "delta", "attention"))
+    return build_engine_from_state_dict(cfg, hybrid_weights(cfg, "cuda"), _engine_config(max_tokens, max_seqs, pages),
+                                        dtype=torch.bfloat16)
+
+
+def vezodra_kernel_table(z: Dict, prefill: int, batch: int, context: int, timer, hbm_gbs: float,
+                         peak_tflops: Dict[str, float]) -> List[Dict]:
+    """Every kernel the Vezodra stack adds or takes in a new form, beside the kernel of the Fomalix (or Pifazen) stack that does
+    the like job (``like``), at prefill (one request) and decode (``batch`` requests) shapes: device time, algorithmic bytes
+    and FLOPs, fraction of the roofline (the larger of bytes / copy bandwidth and FLOPs / the peak of the unit used)."""
+    from .kernels import mixer_ops as M
+    from .kernels import parallel_ops as P
+    from .modules.implementations import DSRotarySinkAttention
+    from .ragged.ragged_wrapper import RaggedBatchWrapper
+    dev, bf = "cuda", torch.bfloat16
+    W, H, G, d, taps, rk = z["width"], z["heads"], z["kv_heads"], z["head"], VEZODRA["taps"], VEZODRA["rank"]
+    n = H * d
+    rows: List[Dict] = []
+
+    def add(name, like, phase, fn, nbytes, flops=0.0, pipe=None):
+        ms = timer(fn, 5, 3)
+        ideal_ms = nbytes / hbm_gbs / 1e6
+        if pipe is not None:
+            ideal_ms = max(ideal_ms, flops / peak_tflops[pipe] / 1e9)
+        rows.append({"kernel": name, "like": like, "phase": phase, "ms": round(ms, 4),
+                     "GB_s": round(nbytes / ms / 1e6, 1), "GFLOP_s": round(flops / ms / 1e6, 1), "pipe": pipe or "memory",
+                     "of_roofline": round(ideal_ms / ms, 3)})
+
+    def randn(*shape, dtype=torch.float32):
+        return torch.randn(*shape, device=dev).to(dtype)
+
+    for phase, T, n_seq, seen in (("prefill", prefill, 1, 0), ("decode", batch, batch, context)):
+        per = T // n_seq
+        tot = seen + per
+        n_pages_seq = (tot + 63) // 64
+        t2s = torch.arange(n_seq, device=dev, dtype=torch.int32).repeat_interleave(per)
+        pos = (torch.arange(per, device=dev, dtype=torch.int32) + seen).repeat(n_seq)
+        tables = torch.arange(n_seq * n_pages_seq, device=dev, dtype=torch.int32).view(n_seq, n_pages_seq)
+        info = torch.tensor([[i * per, per, seen, i] for i in range(n_seq)], dtype=torch.int32, device=dev)
+        single = per == 1
+        # closing a layer (feed-forward + averaged pair) and opening the next (two norms + input filter)
+        x32, y, a, b = randn(T, W), randn(T, W, dtype=bf), randn(T, W, dtype=bf), randn(T, W, dtype=bf)
+        wv = torch.ones(W, device=dev, dtype=bf)
+        filt, fst = randn(taps, W, dtype=bf), torch.zeros(n_seq, taps - 1, W, device=dev)
+        state_bytes = n_seq * (taps - 1) * W * 4 * (2 if seen else 1)
+        for name, part, nb in (("averaged pair + feed-forward", P.StreamSum(y=y, a=a, wa=wv, b=b, wb=wv, mult=0.5), 6),
+                               ("mixer + feed-forward", P.StreamSum(y=y, a=a), 4)):
+            add(f"open_parallel_layer ({name}; two norms, input filter)", None, phase,
+                lambda: P.open_parallel_layer(x32, part, wv, filt, fst, wv, 1e-5, bf, info, t2s, single),
+                T * W * (8 + nb + 4) + state_bytes)
+            add(f"resid_norm_step (post-norm + add + pre-norm), beside {name}",
+                f"open_parallel_layer ({name}; two norms, input filter)", phase,
+                lambda: M.resid_norm_step(x32, y, wv, None, wv, 1e-5, bf), T * W * (4 + 4 + 2 + 2))
+        # attention rows and attention
+        wide = randn(T, (H + 2 * G) * d + 8 * ((H + 7) // 8), dtype=bf)
+        inv = DSRotarySinkAttention.rotary_table(d, 10000.0).to(dev)
+        kc, vc = randn(n_seq * n_pages_seq, 64, G, d, dtype=bf), randn(n_seq * n_pages_seq, 64, G, d, dtype=bf)
+        qn, kn, temp = torch.ones(n, device=dev, dtype=bf), torch.ones(G * d, device=dev, dtype=bf), torch.ones(H, device=dev)
+        row_bytes = T * (H * d * 6 + 2 * G * d * 4)
+        add("rope_append (whole-row norms, halves)", None, phase,
+            lambda: P.rope_append(wide, 0, n, n + G * d, qn, kn, inv, False, None, kc, vc, t2s, pos, tables, H, G, d, d, 1e-5),
+            row_bytes)
+        add("rope_append (interleaved, values from keys, head scale)", None, phase,
+            lambda: P.rope_append(wide, 0, n, n, None, None, inv, True, temp, kc, vc, t2s, pos, tables, H, G, d, d, 1e-5),
+            T * (H * d * 6 + G * d * 6))
+        bias = torch.zeros((H + 2 * G) * d, device=dev, dtype=bf)
+        add("qk_norm_append", "rope_append (whole-row norms, halves)", phase,
+            lambda: M.qk_norm_append(wide, bias, kc, vc, t2s, pos, tables, H, G, d, d, 1e-5, True), row_bytes)
+        wrap = RaggedBatchWrapper(max(T, 64), n_seq, n_pages_seq, device=dev)
+
+        class _Seq:
+            def __init__(self, i):
+                self.seen_tokens, self._b = seen, tables[i].cpu()
+
+            def kv_blocks(self):
+                return self._b
+        for i in range(n_seq):
+            wrap.insert_sequence(_Seq(i), torch.zeros(per, dtype=torch.int32), do_checks=False)
+        wrap.finalize()
+        atoms, n_long = wrap.atoms(), wrap.atoms_longer_than(M.SHORT_ATOM)
+        q32, sink = randn(T, H, d), torch.zeros(H, device=dev)
+        gate = wide[:, (H + 2 * G) * d: (H + 2 * G) * d + H]
+        keys_per_q = (per + 1) / 2 if phase == "prefill" else tot
+        att_bytes, fl = n_seq * tot * 2 * G * d * 2 + T * H * d * 6, 4.0 * T * H * d * keys_per_q
+
+        def attend(**kw):
+            return M.sink_attention(q32, kc, vc, kw.pop("sink", None), t2s, pos, tables, d ** -0.5, kw.pop("chunk", 0), bf, atoms,
+                                    n_long, **kw)
+        add("sink_attention (causal, added one, gate per head)", None, phase, lambda: attend(sink=sink, gate=gate), att_bytes, fl,
+            "fp32")
+        add(f"sink_attention (window {tot})", None, phase, lambda: attend(window=tot), att_bytes, fl, "fp32")
+        chunk = max(CHUNK, tot)
+        add(f"sink_attention (chunk {chunk}, sink)", "sink_attention (causal, added one, gate per head)", phase,
+            lambda: attend(sink=sink, chunk=chunk), att_bytes, fl, "fp32")
+        # delta rule: operands, recurrence, output norm
+        proj = randn(T, 5 * n + rk, dtype=bf)
+        w2, w0 = randn(rk, n, dtype=bf), torch.zeros(n, device=dev)
+        add("removal_prepare (decay, unit key, removal rate; inner projection)", None, phase,
+            lambda: P.removal_prepare(proj, 0, n, 2 * n, 3 * n, 5 * n, w2, w0, w0, H, d, 0.6, 1e-6),
+            T * (n * (4 * 2 + 5 * 4) + rk * 2) + rk * n * 2, 2.0 * T * n * rk, "fp32")
+        b_raw, A_log, dtb = randn(T, 8 * ((H + 7) // 8), dtype=bf), torch.zeros(H, device=dev), torch.zeros(n, device=dev)
+        add("channel_decay_gates", "removal_prepare (decay, unit key, removal rate; inner projection)", phase,
+            lambda: M.channel_decay_gates(proj[:, :n], b_raw[:, :H], A_log, dtb, H, d), T * n * (2 + 4) + T * H * 6)
+        buf = P.removal_prepare(proj, 0, n, 2 * n, 3 * n, 5 * n, w2, w0, w0, H, d, 0.6, 1e-6)
+        S0 = torch.zeros(n_seq, H, d, d, device=dev)
+        sb = n_seq * H * d * d * 4 * (2 if seen else 1)
+        add("removal_recurrence", None, phase, lambda: P.removal_recurrence(buf, S0, info, single), sb + T * n * (5 + 1) * 4,
+            9.0 * T * n * d, "fp32")
+        xs = randn(T, 3 * n)
+        xs[:, : 2 * n] /= math.sqrt(d)
+        decay, beta = torch.rand(T, H, device=dev) * 0.1 + 0.9, torch.rand(T, H, device=dev)
+        add("linear_recurrence (delta, decay per head)", "removal_recurrence", phase,
+            lambda: M.linear_recurrence(xs[:, n: 2 * n], xs[:, :n], xs[:, 2 * n:], decay, beta, None, S0, info, H, H, d, d, True),
+            sb + T * n * 4 * 4, 6.0 * T * n * d, "fp32")
+        o0, gt = randn(T, n), randn(T, n, dtype=bf)
+        add("group_norm_gate (sigmoid gate, one weight per channel)", None, phase,
+            lambda: M.group_norm_gate(o0, gt, qn, d, 1e-5, False, bf, sigmoid=True), T * n * 8)
+        nw = torch.ones(d, device=dev, dtype=bf)
+        add("group_norm_gate (silu gate, weight shared by the heads)", "group_norm_gate (sigmoid gate, one weight per channel)",
+            phase, lambda: M.group_norm_gate(o0, gt, nw, d, 1e-5, False, bf), T * n * 8)
+    by_name = {(r_["kernel"], r_["phase"]): r_ for r_ in rows}
+    for r_ in rows:                      # distance from the roofline relative to the like kernel's
+        if r_["like"]:
+            mine = by_name[(r_["like"], r_["phase"])]
+            mine["like_of_roofline"], mine["like_kernel"] = r_["of_roofline"], r_["kernel"]
+    return rows
+
+
 def run(sizes: List[str], prefill: int, batch: int, context: int, steps: int, warmup: int, kernels: bool = True,
         chunk: int = 0, model: str = "fomalix") -> Dict:
     global CHUNK, WINDOW
@@ -987,6 +1175,21 @@ def run(sizes: List[str], prefill: int, batch: int, context: int, steps: int, wa
                      "kekopel": engine_throughput(build_kekopel, z, prefill, batch, context, steps, warmup, timer)}
             if kernels:
                 entry["kernels"] = pifazen_kernel_table(z, prefill, batch, context, timer, hbm, peak_tflops)
+            out["sizes"][name] = entry
+        return out
+    if model == "vezodra":
+        out["metric"] = "serving tokens/s, Vezodra vs a Fomalix stack of attention and delta-rule layers of equal size"
+        out["vezodra"] = VEZODRA
+        WINDOW = CHUNK = max(WINDOW, prefill, context + steps + warmup + 8)    # window and chunk hold every key: equal work
+        out["attention_window"] = out["attention_chunk"] = WINDOW
+        for name in sizes:
+            z = SIZES[name]
+            entry = {"config": z,
+                     "vezodra": engine_throughput(build_vezodra, z, prefill, batch, context, steps, warmup, timer),
+                     "fomalix_attention_delta": engine_throughput(build_attention_delta_stack, z, prefill, batch, context, steps,
+                                                                  warmup, timer)}
+            if kernels:
+                entry["kernels"] = vezodra_kernel_table(z, prefill, batch, context, timer, hbm, peak_tflops)
             out["sizes"][name] = entry
         return out
     if model == "ridazen":
