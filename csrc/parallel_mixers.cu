@@ -232,11 +232,26 @@ norm_filter_vec_kernel(const float* __restrict__ x, const float* __restrict__ rs
     for (int e = 0; e < 8; ++e) h[e] *= r * w1v[e];
   };
   bool need = true;
+  int first = 0, end = 0;                                // the current sequence's rows in the batch
+  const int* si = seq_info;
+  float nx[8], nr = rstd[t0];                            // the next row, fetched one row ahead
+  load8_f32<float>(x + (long long)t0 * C + c0, nx);
   for (int t = t0; t < n_tokens; ++t) {
-    const int* si = seq_info + 4 * tok_seq[t];
-    const int first = si[0], local = t - first;
+    if (t >= end) {
+      si = seq_info + 4 * tok_seq[t];
+      first = si[0], end = first + si[1];
+    }
+    const int local = t - first;
     const bool head = local > 0 && local < KEEP;         // belongs to the thread of the sequence's first row
     if (t >= t1 && !(head && first >= t0)) break;
+    float xv[8], o[8];
+    const float r = nr;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) xv[e] = nx[e];
+    if (t + 1 < n_tokens) {
+      load8_f32<float>(x + (long long)(t + 1) * C + c0, nx);
+      nr = rstd[t + 1];
+    }
     if (head && first < t0) continue;
     if (local == 0) {
       const int n = si[1], seen = si[2];
@@ -278,9 +293,6 @@ norm_filter_vec_kernel(const float* __restrict__ x, const float* __restrict__ rs
         for (int e = 0; e < 8; ++e) hist[j][e] = hist[j - 1][e];
     }
     need = false;
-    float xv[8], o[8];
-    load8_f32<float>(x + (long long)t * C + c0, xv);
-    const float r = rstd[t];
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
       xv[e] *= r;
