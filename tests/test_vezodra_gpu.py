@@ -1,6 +1,5 @@
 """The Vezodra cases of ``test_vezodra.py`` on the CUDA kernels (``csrc/parallel_mixers.cu``, ``csrc/seq_mixers.cu``): the same
 functions, collected here under the ``gpu`` marker; the ops take their kernel branch because their tensors live on the device."""
-import math
 
 import pytest
 import torch
@@ -77,3 +76,27 @@ def test_wide_streams():
     from test_vezodra import test_sums_norms_and_input_filter as case
     for W, taps in ((8200, 4), (4096, 4), (8192, 3), (1001, 2)):
         case(W, taps, True)
+
+
+def test_queued_batches_never_share_a_staging_buffer():
+    """Forwards are queued without a synchronisation: while a long kernel holds the stream back, later batches must not
+    overwrite the metadata of the uploads that still wait behind it."""
+    from shuffle_exchange_b200.inference.v2.ragged.ragged_wrapper import RaggedBatchWrapper
+
+    class _Seq:
+        seen_tokens = 0
+
+        def kv_blocks(self):
+            return torch.zeros(1, dtype=torch.int32)
+    wrap = RaggedBatchWrapper(16, 2, 4, device="cuda")
+    big = torch.randn(4096, 4096, device="cuda")
+    for _ in range(20):
+        big = big @ big / 64.0
+    got = []
+    for i in range(3):
+        wrap.clear()
+        wrap.insert_sequence(_Seq(), torch.full((5,), 100 + i, dtype=torch.int32))
+        wrap.finalize()
+        got.append(wrap.input_ids().clone())
+    torch.cuda.synchronize()
+    assert [int(g[0]) for g in got] == [100, 101, 102] and all(bool((g == g[0]).all()) for g in got)
