@@ -93,16 +93,18 @@ top_k_gating_kernel(const T* __restrict__ logits, float* __restrict__ scores, in
 }
 
 // Group-limited gating with a choice correction, one warp per token.  Scores are the softmax over all E router outputs
-// (fp32); the CHOICE is made by score + correction: the experts form n_groups contiguous blocks of equal size, a group's rank
-// is the largest choice value in it, only members of the keep_groups best groups can win, and the top_k largest choice
-// values among them are taken.  The weights are the winners' plain scores (no correction), normalised by their total plus 1e-20
-// and multiplied by `scale`.  Outputs as top_k_gating_kernel.
+// (fp32), or the sigmoid of each (kScoreSigmoid); the CHOICE is made by score + correction: the experts form n_groups
+// contiguous blocks of equal size, a group's rank is the largest choice value in it (kRankTopTwo: the sum of its two largest),
+// only members of the keep_groups best groups can win, and the top_k largest choice values among them are taken.  The weights
+// are the winners' plain scores (no correction), normalised by their total plus 1e-20 (kPlainWeights: as they are) and
+// multiplied by `scale`.  Outputs as top_k_gating_kernel.
+constexpr int kScoreSigmoid = 1, kRankTopTwo = 2, kPlainWeights = 4;
 constexpr int kMaxGroups = 128;
 __global__ void __launch_bounds__(256)
 grouped_top_k_gating_kernel(const float* __restrict__ logits, const float* __restrict__ correction,
                             float* __restrict__ scores, int* __restrict__ assignments, int* __restrict__ offsets,
                             int* __restrict__ expert_counts, int n_tokens, int n_experts, int top_k, int n_groups,
-                            int keep_groups, float scale) {
+                            int keep_groups, float scale, int flags) {
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   const int lane = threadIdx.x & 31;
   if (warp >= n_tokens) return;
@@ -116,15 +118,20 @@ grouped_top_k_gating_kernel(const float* __restrict__ logits, const float* __res
     p[i] = (e < n_experts) ? row[e] : -INFINITY;
     mx = fmaxf(mx, p[i]);
   }
-  mx = warp_max(mx);
-  float sum = 0.f;
+  float inv = 1.f;
+  if (flags & kScoreSigmoid) {
 #pragma unroll
-  for (int i = 0; i < PER; ++i) {
-    p[i] = (i * 32 + lane < n_experts) ? expf(p[i] - mx) : 0.f;
-    sum += p[i];
+    for (int i = 0; i < PER; ++i) p[i] = (i * 32 + lane < n_experts) ? 1.f / (1.f + expf(-p[i])) : 0.f;
+  } else {
+    mx = warp_max(mx);
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      p[i] = (i * 32 + lane < n_experts) ? expf(p[i] - mx) : 0.f;
+      sum += p[i];
+    }
+    inv = 1.f / warp_sum(sum);
   }
-  sum = warp_sum(sum);
-  const float inv = 1.f / sum;
   const int per_group = n_experts / n_groups;
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
@@ -138,13 +145,22 @@ grouped_top_k_gating_kernel(const float* __restrict__ logits, const float* __res
 #pragma unroll
     for (int j = 0; j < PERG; ++j) gmax[j] = -INFINITY;
     for (int g = 0; g < n_groups; ++g) {
-      float m = -INFINITY;
+      float m = -INFINITY, m2 = -INFINITY;              // the group's largest and second largest choice value
 #pragma unroll
       for (int i = 0; i < PER; ++i) {
         const int e = i * 32 + lane;
-        if (e < n_experts && e / per_group == g) m = fmaxf(m, ch[i]);
+        if (e < n_experts && e / per_group == g) m2 = fmaxf(m2, fminf(m, ch[i])), m = fmaxf(m, ch[i]);
       }
-      m = warp_max(m);
+      if (flags & kRankTopTwo) {
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+          const float om = __shfl_xor_sync(0xffffffffu, m, o), om2 = __shfl_xor_sync(0xffffffffu, m2, o);
+          m2 = fmaxf(fminf(m, om), fmaxf(m2, om2)), m = fmaxf(m, om);
+        }
+        if (per_group > 1) m += m2;
+      } else {
+        m = warp_max(m);
+      }
 #pragma unroll
       for (int j = 0; j < PERG; ++j)
         if (j * 32 + lane == g) gmax[j] = m;
@@ -213,7 +229,7 @@ grouped_top_k_gating_kernel(const float* __restrict__ logits, const float* __res
     picked_sum += best_p;
   }
   if (lane == 0) {
-    const float norm = scale / (picked_sum + 1e-20f);
+    const float norm = (flags & kPlainWeights) ? scale : scale / (picked_sum + 1e-20f);
     for (int k = 0; k < top_k; ++k) {
       const long long o = (long long)warp * top_k + k;
       scores[o] = my_score[k] * norm;
@@ -575,10 +591,12 @@ SXB_API int sxb_top_k_gating(const void* logits, void* scores, void* assignments
 // Group-limited gating with a choice correction.  logits fp32 [T, E]; correction fp32 [E] or null; the E experts form
 // n_groups contiguous blocks of equal size of which the keep_groups whose best (score + correction) is largest stay eligible;
 // the top_k largest (score + correction) among them win; scores fp32 [T, K] = softmax score of the winner / (sum of the
-// winners' scores + 1e-20) * scale; assignments / offsets / expert_counts as sxb_top_k_gating.
+// winners' scores + 1e-20) * scale; assignments / offsets / expert_counts as sxb_top_k_gating.  flags: 1 = the score is the
+// sigmoid of the expert's own logit, 2 = groups are ranked by the sum of their two largest (score + correction), 4 = the
+// winners' scores are not divided by their sum.
 SXB_API int sxb_grouped_top_k_gating(const void* logits, const void* correction, void* scores, void* assignments,
                                      void* offsets, void* expert_counts, int n_tokens, int n_experts, int top_k,
-                                     int n_groups, int keep_groups, float scale, void* stream) {
+                                     int n_groups, int keep_groups, float scale, int flags, void* stream) {
   if (n_tokens <= 0) return SXB_OK;
   if (n_experts <= 0 || n_experts > moe::kMaxExperts || top_k <= 0 || top_k > moe::kMaxTopK || top_k > n_experts)
     return SXB_ERR_BAD_ARG;
@@ -590,7 +608,7 @@ SXB_API int sxb_grouped_top_k_gating(const void* logits, const void* correction,
   moe::grouped_top_k_gating_kernel<<<(unsigned)((n_tokens + 7) / 8), 256, 0, s>>>(
       static_cast<const float*>(logits), static_cast<const float*>(correction), static_cast<float*>(scores),
       static_cast<int*>(assignments), static_cast<int*>(offsets), static_cast<int*>(expert_counts), n_tokens, n_experts,
-      top_k, n_groups, keep_groups, scale);
+      top_k, n_groups, keep_groups, scale, flags);
   SXB_CHECK_LAUNCH();
   return SXB_OK;
 }

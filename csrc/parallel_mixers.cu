@@ -357,7 +357,7 @@ norm_filter_state_kernel(const float* __restrict__ x, const float* __restrict__ 
 // One CTA per token.  q (Hq d channels at column q0), k (G d at k0) and v (G dv at v0; v0 may be k0: the values are then the
 // projected keys as they are) of a fused projection row.  q_w / k_w (Hq d / G d entries): the WHOLE row of q / of k is divided by
 // its root mean square and multiplied by the weight.  The first n_rot channels of every head turn by pos * inv_freq[i] in
-// pairs (2i, 2i+1) (interleaved) or (i, i + n_rot/2).  q -> fp32 [tokens, Hq, d], times q_scale[h]; k, v -> paged caches.
+// pairs (2i, 2i+1) (interleaved) or (i, i + n_rot/2), cos and sin times amp.  q -> fp32 [tokens, Hq, d], times q_scale[h]; k, v -> paged caches.
 // VEC 4: all columns, sizes and the rotated part's pieces are multiples of 4 channels.
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
@@ -365,14 +365,19 @@ rope_append_kernel(const T* __restrict__ proj, long long ld, int q0, int k0, int
                    const T* __restrict__ k_w, const float* __restrict__ inv_freq, const float* __restrict__ q_scale,
                    float* __restrict__ q_out, T* __restrict__ kcache, T* __restrict__ vcache,
                    const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, const int* __restrict__ tables,
-                   int max_blocks, int block_size, int Hq, int G, int d, int dv, int n_rot, int interleaved, float eps) {
+                   int max_blocks, int block_size, int Hq, int G, int d, int dv, int n_rot, int interleaved, float eps,
+                   float amp) {
   extern __shared__ __align__(16) float cs[];   // cos [n_rot / 2] | sin [n_rot / 2]
   __shared__ float2 red[32];
   const int t = blockIdx.x, half = n_rot >> 1;
   const T* row = proj + (long long)t * ld;
   const int pos = tok_pos[t];
   const long long slot = (long long)tables[(long long)tok_seq[t] * max_blocks + pos / block_size] * block_size + pos % block_size;
-  for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)pos * inv_freq[i], &cs[half + i], &cs[i]);
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float sn, co;
+    sincosf((float)pos * inv_freq[i], &sn, &co);
+    cs[i] = co * amp, cs[half + i] = sn * amp;
+  }
   float iq = 1.f, ik = 1.f;
   if (q_w != nullptr || k_w != nullptr) {
     float sq = 0.f, sk = 0.f;
@@ -873,14 +878,15 @@ SXB_API int sxb_norm_filter_rows(const void* x, const void* rstd, const void* w1
 
 /* Rows of a fused projection (`dtype`, pitch ld): q (Hq d channels at column q0), k (G d at k0), v (G dv at v0, which may be k0).
  * q_w / k_w (`dtype` [Hq d] / [G d] or null): RMS norm over the whole row of q / k with that weight.  The first n_rot channels of
- * every q and k head turn by pos * inv_freq[i] (fp32 [n_rot / 2]) in pairs (2i, 2i+1) (interleaved != 0) or (i, i + n_rot/2).
+ * every q and k head turn by pos * inv_freq[i] (fp32 [n_rot / 2]) in pairs (2i, 2i+1) (interleaved != 0) or (i, i + n_rot/2), cos
+ * and sin multiplied by amp.
  * q -> q_out fp32 [n_tokens, Hq, d] times q_scale[h] (fp32 or null), k -> kcache [pages, block_size, G, d], v -> vcache
  * [pages, block_size, G, dv] at each token's (page, offset). */
 SXB_API int sxb_rope_append(const void* proj, long long ld, int q0, int k0, int v0, const void* q_w, const void* k_w,
                             const void* inv_freq, const void* q_scale, void* q_out, void* kcache, void* vcache,
                             const void* tok_seq, const void* tok_pos, const void* tables, int n_tokens, int max_blocks,
-                            int block_size, int Hq, int G, int d, int dv, int n_rot, int interleaved, float eps, int dtype,
-                            void* stream) {
+                            int block_size, int Hq, int G, int d, int dv, int n_rot, int interleaved, float eps, float amp,
+                            int dtype, void* stream) {
   if (n_tokens <= 0) return SXB_OK;
   if (n_rot < 0 || n_rot > d || (n_rot & 1) || (n_rot > 0 && inv_freq == nullptr) || Hq % G) return SXB_ERR_BAD_ARG;
   const int turn = interleaved ? n_rot : n_rot / 2;
@@ -893,7 +899,7 @@ SXB_API int sxb_rope_append(const void* proj, long long ld, int q0, int k0, int 
                              (const T*)proj, ld, q0, k0, v0, (const T*)q_w, (const T*)k_w, (const float*)inv_freq,     \
                              (const float*)q_scale, (float*)q_out, (T*)kcache, (T*)vcache, (const int*)tok_seq,        \
                              (const int*)tok_pos, (const int*)tables, max_blocks, block_size, Hq, G, d, dv, n_rot,     \
-                             interleaved, eps)))
+                             interleaved, eps, amp)))
   if (vec) ROPE_APPEND(4);
   else ROPE_APPEND(1);
 #undef ROPE_APPEND

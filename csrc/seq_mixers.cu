@@ -48,15 +48,15 @@ embed_sinusoid_kernel(const int* __restrict__ ids, const int* __restrict__ pos, 
 }
 
 // ------------------------------------------------------------------------------------------------ residual + norms
-// One CTA per row.  y (optional): residual += mult * y / rms(y) * w_post, or += mult * y without w_post; with y_scale
-// the addend is also multiplied per channel by y_scale.  extra (optional): residual += extra.  w_pre (optional):
-// out = residual / rms(residual) * (w_add + w_pre) (w_add 1 for weights stored as their distance from one); out without
-// w_pre: the residual itself in the activation type.
+// One CTA per row.  y (optional): residual += mult * y / rms(y) * (post_add + w_post), or += mult * y without w_post; with
+// y_scale the addend is also multiplied per channel by y_scale.  extra (optional): residual += extra.  w_pre (optional):
+// out = residual / rms(residual) * (w_add + w_pre) (w_add, post_add 1 for weights stored as their distance from one); out
+// without w_pre: the residual itself in the activation type.
 template <typename T>
 __global__ void __launch_bounds__(256)
 resid_norm_step_kernel(float* __restrict__ resid, const T* __restrict__ y, const T* __restrict__ w_post,
                        const float* __restrict__ extra, const T* __restrict__ w_pre, T* __restrict__ out, int width,
-                       float eps, float mult, const T* __restrict__ y_scale, float w_add) {
+                       float eps, float mult, const T* __restrict__ y_scale, float w_add, float post_add) {
   __shared__ float red[32];
   const long long base = (long long)blockIdx.x * width;
   float* r = resid + base;
@@ -74,7 +74,7 @@ resid_norm_step_kernel(float* __restrict__ resid, const T* __restrict__ y, const
   for (int c = threadIdx.x; c < width; c += blockDim.x) {
     float v = r[c];
     if (y != nullptr) {
-      float add = to_f32<T>(y[base + c]) * inv_y * (w_post ? to_f32<T>(w_post[c]) : 1.f);
+      float add = to_f32<T>(y[base + c]) * inv_y * (w_post ? post_add + to_f32<T>(w_post[c]) : 1.f);
       if (y_scale != nullptr) add *= to_f32<T>(y_scale[c]);
       v += add;
     }
@@ -91,6 +91,62 @@ resid_norm_step_kernel(float* __restrict__ resid, const T* __restrict__ y, const
   const float inv = 1.f / sqrtf(ss2 / (float)width + eps);
   for (int c = threadIdx.x; c < width; c += blockDim.x)
     out[base + c] = from_f32<T>(r[c] * inv * (w_add + to_f32<T>(w_pre[c])));
+}
+
+// The same with the row in registers, eight consecutive channels per thread (16-byte accesses): widths that are multiples of
+// 8 up to 8192, blockDim.x * 8 >= width.
+template <typename T>
+__global__ void __launch_bounds__(1024)
+resid_norm_step_vec_kernel(float* __restrict__ resid, const T* __restrict__ y, const T* __restrict__ w_post,
+                           const float* __restrict__ extra, const T* __restrict__ w_pre, T* __restrict__ out, int width,
+                           float eps, float mult, const T* __restrict__ y_scale, float w_add, float post_add) {
+  __shared__ float red[32];
+  const int c0 = threadIdx.x * 8;
+  const bool live = c0 < width;
+  const long long at = (long long)blockIdx.x * width + c0;
+  float x[8], v[8], w[8];
+#pragma unroll
+  for (int e = 0; e < 8; ++e) x[e] = v[e] = 0.f;
+  if (live) load8_f32<float>(resid + at, x);
+  if (y != nullptr) {
+    if (live) load8_f32<T>(y + at, v);
+    float inv = mult;
+    if (w_post != nullptr) {
+      float ss = 0.f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss += v[e] * v[e];
+      if (live) load8_f32<T>(w_post + c0, w);
+      inv = mult / sqrtf(block_sum(ss, red) / (float)width + eps);
+    }
+    if (live) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] *= inv * (w_post ? post_add + w[e] : 1.f);
+      if (y_scale != nullptr) {
+        load8_f32<T>(y_scale + c0, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] *= w[e];
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] += v[e];
+    }
+  }
+  if (extra != nullptr && live) {
+    load8_f32<float>(extra + at, v);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[e] += v[e];
+  }
+  if ((y != nullptr || extra != nullptr) && live) store8_f32<float>(resid + at, x);
+  if (out == nullptr) return;
+  if (w_pre != nullptr) {
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss += x[e] * x[e];
+    if (live) load8_f32<T>(w_pre + c0, w);
+    const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)width + eps);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[e] *= inv * (w_add + w[e]);
+  }
+  if (live) store8_f32<T>(out + at, x);
 }
 
 // ------------------------------------------------------------------------------------------------ attention
@@ -137,8 +193,10 @@ qk_norm_append_kernel(const T* __restrict__ qkv, long long ld, const T* __restri
 // and the row pitch allow.  Every channel of q | k | v is filtered over time (w [C, taps], last tap = current token;
 // earlier inputs from this batch's rows, else from the slot's carried inputs state [slots, taps-1, C], else zero; w null:
 // no filter), q and k heads are divided by their root mean square and multiplied by a weight of d entries that all
-// heads share (null: none), and q by 1 + coef * ln(floor((pos + 1) / every) + 1).  Filter sums, norms and the
-// temperature are fp32.
+// heads share (null: none), and q by 1 + coef * ln(floor((pos + 1) / every) + 1).  Then the first n_rot channels of every q
+// and k head turn by pos * inv_freq[i] in pairs (i, i + n_rot/2) or, interleaved, (2i, 2i+1), cos and sin times amp: the
+// CTA's four warps share the angles of its rows, and a warp passes its head through shared memory so that every lane finds
+// the other channel of its pairs.  Filter sums, norms, angles and the temperature are fp32.
 template <typename T, int VEC>
 struct alignas(sizeof(T) * VEC) Pack {
   T v[VEC];
@@ -181,9 +239,21 @@ qkv_filter_norm_append_kernel(const T* __restrict__ qkv, long long ld, const T* 
                               T* __restrict__ kcache, T* __restrict__ vcache, const int* __restrict__ tok_seq,
                               const int* __restrict__ tok_pos, const int* __restrict__ tables, int max_blocks,
                               int block_size, int Hq, int G, int d, int dv, int taps, float eps, int normalize,
-                              float temp_coef, int temp_every, int vec_ok, int n_tokens, int rows_per_warp) {
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+                              float temp_coef, int temp_every, int vec_ok, int n_tokens, int rows_per_warp,
+                              const float* __restrict__ inv_freq, int n_rot, int interleaved, float amp) {
+  extern __shared__ __align__(16) float turn[];      // n_rot > 0: [rows_per_warp][cos (half) | sin (half)], [4 warps][32 VEC]
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = n_rot >> 1;
   const int s = blockIdx.y * 4 + warp;
+  if (n_rot > 0) {
+    for (int i = threadIdx.x; i < rows_per_warp * half; i += blockDim.x) {
+      const int r = i / half, p = i % half, t = blockIdx.x * rows_per_warp + r;
+      if (t >= n_tokens) break;
+      float sn, cs;
+      sincosf((float)tok_pos[t] * inv_freq[p], &sn, &cs);
+      turn[r * n_rot + p] = cs * amp, turn[r * n_rot + half + p] = sn * amp;
+    }
+    __syncthreads();
+  }
   if (s >= Hq + 2 * G) return;
   const int C = (Hq + G) * d + G * dv;
   const bool is_v = s >= Hq + G;
@@ -262,10 +332,28 @@ qkv_filter_norm_append_kernel(const T* __restrict__ qkv, long long ld, const T* 
       if (normalize) inv = 1.f / sqrtf(ss / (float)d + eps);
       if (s < Hq && temp_coef != 0.f) inv *= 1.f + temp_coef * logf((float)((pos + 1) / temp_every + 1));
     }
-    if (valid <= 0) continue;
     float o[VEC];
 #pragma unroll
     for (int i = 0; i < VEC; ++i) o[i] = v[i] * inv * gain[i];
+    if (n_rot > 0 && !is_v) {
+      float* mine = turn + rows_per_warp * n_rot + warp * 32 * VEC;
+      const float* cs = turn + (t - t0) * n_rot;
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) mine[c0 + i] = o[i];
+      __syncwarp();
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) {
+        const int c = c0 + i;
+        if (c < n_rot) {
+          const int p = interleaved ? c >> 1 : (c < half ? c : c - half);
+          const bool first = interleaved ? !(c & 1) : c < half;
+          const float other = mine[interleaved ? c ^ 1 : (first ? c + half : c - half)];
+          o[i] = first ? o[i] * cs[p] - other * cs[half + p] : o[i] * cs[p] + other * cs[half + p];
+        }
+      }
+      __syncwarp();
+    }
+    if (valid <= 0) continue;
     if (s < Hq) {
       store_pack<float, VEC>(q_out + ((long long)t * Hq + s) * d + c0, o, vec, valid);
     } else {
@@ -300,7 +388,7 @@ sink_attention_tile_kernel(const float* __restrict__ q, const T* __restrict__ kc
                            const int* __restrict__ tables, int max_blocks, int block_size, int Hq, int G, int d,
                            int dv, float scale, int chunk, int window, int kpitch, int vpitch,
                            const float* __restrict__ dist_bias, int bias_len, const T* __restrict__ gate,
-                           long long gate_ld, int gate_heads) {
+                           long long gate_ld, int gate_heads, long long out_ld, float out_scale) {
   extern __shared__ __align__(16) float smf[];
   const int dp = d + 4, vp = NV * 64, pp = kBK + 4;
   float* Qs = smf;
@@ -447,7 +535,7 @@ sink_attention_tile_kernel(const float* __restrict__ q, const T* __restrict__ kc
         if (c < dv) {
           float o = ((e & 1) ? a2.y : a2.x) * inv;
           if (gate != nullptr) o *= sigmoid_f(to_f32<T>(gate[(long long)(row0 + r) * gate_ld + (gate_heads ? h : h * dv + c)]));
-          out[((long long)(row0 + r) * Hq + h) * dv + c] = from_f32<T>(o);
+          out[(long long)(row0 + r) * out_ld + h * dv + c] = from_f32<T>(o * out_scale);
         }
       }
   }
@@ -488,7 +576,7 @@ sink_attention_kernel(const float* __restrict__ q, const T* __restrict__ kcache,
                       const int* __restrict__ tok_pos, const int* __restrict__ tables, int max_blocks, int block_size,
                       int Hq, int G, int d, int dv, float scale, int chunk, int window, int kpitch, int vpitch,
                       const int* __restrict__ atoms, const float* __restrict__ dist_bias, int bias_len,
-                      const T* __restrict__ gate, long long gate_ld, int gate_heads) {
+                      const T* __restrict__ gate, long long gate_ld, int gate_heads, long long out_ld, float out_scale) {
   // q [REP][d8] | partial values [kAW][REP][dv] | partial max [kAW][REP] | partial sum [kAW][REP] | key staging
   extern __shared__ __align__(16) float qs[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -648,7 +736,7 @@ sink_attention_kernel(const float* __restrict__ q, const T* __restrict__ kcache,
     }
     float r = L > 0.f ? o / L : 0.f;
     if (gate != nullptr) r *= sigmoid_f(to_f32<T>(gate[(long long)t * gate_ld + (gate_heads ? h0 + hh : (h0 + hh) * dv + c)]));
-    out[((long long)t * Hq + h0 + hh) * dv + c] = from_f32<T>(r);
+    out[(long long)t * out_ld + (h0 + hh) * dv + c] = from_f32<T>(r * out_scale);
   }
 }
 
@@ -657,7 +745,8 @@ static int launch_attention_rows_v(dim3 grid, const void* q, const void* kcache,
                                    void* out, const void* tok_seq, const void* tok_pos, const void* tables,
                                    int max_blocks, int block_size, int Hq, int G, int d, int dv, float scale,
                                    int chunk, int window, int kpitch, int vpitch, const int* atoms, const void* dist_bias,
-                                   int bias_len, const void* gate, long long gate_ld, int gate_heads, cudaStream_t s) {
+                                   int bias_len, const void* gate, long long gate_ld, int gate_heads, long long out_ld,
+                                   float out_scale, cudaStream_t s) {
   const size_t smem = (size_t)(REP * ((d + 7) & ~7) + kAW * REP * dv + 2 * kAW * REP + kAW * 32 * 68) * sizeof(float);
   cudaError_t e = cudaFuncSetAttribute(sink_attention_kernel<T, REP, VPL>,
                                        cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -666,7 +755,7 @@ static int launch_attention_rows_v(dim3 grid, const void* q, const void* kcache,
   sink_attention_kernel<T, REP, VPL><<<grid, 32 * kAW, smem, s>>>(
       (const float*)q, (const T*)kcache, (const T*)vcache, (const float*)sink, (T*)out, (const int*)tok_seq,
       (const int*)tok_pos, (const int*)tables, max_blocks, block_size, Hq, G, d, dv, scale, chunk, window, kpitch,
-      vpitch, atoms, (const float*)dist_bias, bias_len, (const T*)gate, gate_ld, gate_heads);
+      vpitch, atoms, (const float*)dist_bias, bias_len, (const T*)gate, gate_ld, gate_heads, out_ld, out_scale);
   return SXB_OK;
 }
 
@@ -675,14 +764,15 @@ static int launch_attention_rows(dim3 grid, const void* q, const void* kcache, c
                                  void* out, const void* tok_seq, const void* tok_pos, const void* tables,
                                  int max_blocks, int block_size, int Hq, int G, int d, int dv, float scale, int chunk,
                                  int window, int kpitch, int vpitch, const int* atoms, const void* dist_bias,
-                                 int bias_len, const void* gate, long long gate_ld, int gate_heads, cudaStream_t s) {
+                                 int bias_len, const void* gate, long long gate_ld, int gate_heads, long long out_ld,
+                                   float out_scale, cudaStream_t s) {
   if (dv <= 128)
     return launch_attention_rows_v<T, REP, 4>(grid, q, kcache, vcache, sink, out, tok_seq, tok_pos, tables, max_blocks,
                                               block_size, Hq, G, d, dv, scale, chunk, window, kpitch, vpitch, atoms,
-                                              dist_bias, bias_len, gate, gate_ld, gate_heads, s);
+                                              dist_bias, bias_len, gate, gate_ld, gate_heads, out_ld, out_scale, s);
   return launch_attention_rows_v<T, REP, kMaxVPerLane>(grid, q, kcache, vcache, sink, out, tok_seq, tok_pos, tables,
                                                        max_blocks, block_size, Hq, G, d, dv, scale, chunk, window,
-                                                       kpitch, vpitch, atoms, dist_bias, bias_len, gate, gate_ld, gate_heads, s);
+                                                       kpitch, vpitch, atoms, dist_bias, bias_len, gate, gate_ld, gate_heads, out_ld, out_scale, s);
 }
 
 // Query heads per key/value head that one CTA takes together: the largest of 8, 4, 2, 1 that divides the group.
@@ -690,7 +780,8 @@ static int attention_rows(int dtype, dim3 grid, const void* q, const void* kcach
                           const void* sink, void* out, const void* tok_seq, const void* tok_pos, const void* tables,
                           int max_blocks, int block_size, int Hq, int G, int d, int dv, float scale, int chunk,
                           int window, int kpitch, int vpitch, const int* atoms, const void* dist_bias, int bias_len,
-                          const void* gate, long long gate_ld, int gate_heads, cudaStream_t s) {
+                          const void* gate, long long gate_ld, int gate_heads, long long out_ld,
+                                   float out_scale, cudaStream_t s) {
   const int group = Hq / G;
   int rc = SXB_OK;
   // (Taking fewer heads together when a decode batch leaves SMs idle was measured slower: every CTA walks all keys.)
@@ -699,7 +790,7 @@ static int attention_rows(int dtype, dim3 grid, const void* q, const void* kcach
   SEQMIX_DISPATCH(dtype, (rc = launch_attention_rows<T, REP>(grid, q, kcache, vcache, sink, out, tok_seq, tok_pos,      \
                                                               tables, max_blocks, block_size, Hq, G, d, dv, scale,      \
                                                               chunk, window, kpitch, vpitch, atoms, dist_bias,      \
-                                                              bias_len, gate, gate_ld, gate_heads, s)))
+                                                              bias_len, gate, gate_ld, gate_heads, out_ld, out_scale, s)))
   if (rep == 8) ROWS(8);
   else if (rep == 4) ROWS(4);
   else if (rep == 2) ROWS(2);
@@ -711,27 +802,28 @@ static int attention_rows(int dtype, dim3 grid, const void* q, const void* kcach
 // ------------------------------------------------------------------------------------------------ short convolution
 constexpr int kMaxTaps = 16;
 
-// out[t, c] = silu(bias[c] + sum_j w[c, taps-1-j] * x[t-j, c]); x before this batch's rows comes from the slot's carried
-// inputs (state [slots, taps-1, C], last row = most recent), x before the sequence's start is zero.
+// out[t, c] = act(bias[c] + sum_j w[c, taps-1-j] * (x[t-j, c] + in_bias[c])), act SiLU or none; x before this batch's rows comes
+// from the slot's carried inputs (state [slots, taps-1, C], last row = most recent), terms before the sequence's start are zero.
 template <typename T>
 __global__ void __launch_bounds__(256)
 conv_silu_kernel(const T* __restrict__ x, long long ld, const T* __restrict__ w, const T* __restrict__ bias,
                  const T* __restrict__ state, const int* __restrict__ seq_info, const int* __restrict__ tok_seq,
-                 float* __restrict__ out, int C, int taps) {
+                 float* __restrict__ out, int C, int taps, const T* __restrict__ in_bias, int act) {
   const int t = blockIdx.x;
   const int* si = seq_info + 4 * tok_seq[t];
   const int local = t - si[0], seen = si[2];
   const T* st = state + (long long)si[3] * (taps - 1) * C;
   for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x) {
     float a = bias ? to_f32<T>(bias[c]) : 0.f;
+    const float ib = in_bias ? to_f32<T>(in_bias[c]) : 0.f;
     for (int j = 0; j < taps; ++j) {
       const int src = local - j;
       float v = 0.f;
-      if (src >= 0) v = to_f32<T>(x[(long long)(t - j) * ld + c]);
-      else if (seen + src >= 0) v = to_f32<T>(st[(long long)(taps - 1 + src) * C + c]);
+      if (src >= 0) v = to_f32<T>(x[(long long)(t - j) * ld + c]) + ib;
+      else if (seen + src >= 0) v = to_f32<T>(st[(long long)(taps - 1 + src) * C + c]) + ib;
       a += to_f32<T>(w[(long long)c * taps + (taps - 1 - j)]) * v;
     }
-    out[(long long)t * C + c] = silu_f(a);
+    out[(long long)t * C + c] = act ? silu_f(a) : a;
   }
 }
 
@@ -745,14 +837,15 @@ template <typename T, int TAPS>
 __global__ void __launch_bounds__(128)
 conv_silu_vec_kernel(const T* __restrict__ x, long long ld, const T* __restrict__ w, const T* __restrict__ bias,
                      const T* __restrict__ state, const int* __restrict__ seq_info, const int* __restrict__ tok_seq,
-                     float* __restrict__ out, int C, int n_tokens) {
+                     float* __restrict__ out, int C, int n_tokens, const T* __restrict__ in_bias, int act) {
   const int c0 = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
   if (c0 >= C) return;
   const int t0 = blockIdx.x * kConvRows, t1 = min(t0 + kConvRows, n_tokens);
-  float wt[8][TAPS], b8[8], hist[TAPS][8];      // hist[j]: the input j rows back (hist[0]: the current row)
+  float wt[8][TAPS], b8[8], ib[8], hist[TAPS][8];      // hist[j]: the input j rows back (hist[0]: the current row)
 #pragma unroll
   for (int e = 0; e < 8; ++e) {
     b8[e] = bias ? to_f32<T>(bias[c0 + e]) : 0.f;
+    ib[e] = in_bias ? to_f32<T>(in_bias[c0 + e]) : 0.f;
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) wt[e][j] = to_f32<T>(w[(long long)(c0 + e) * TAPS + j]);
   }
@@ -766,8 +859,12 @@ conv_silu_vec_kernel(const T* __restrict__ x, long long ld, const T* __restrict_
         const int src = local - j;
         if (src >= 0) {
           load8_f32<T>(x + (long long)(t - j) * ld + c0, hist[j]);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) hist[j][e] += ib[e];
         } else if (seen + src >= 0) {
           load8_f32<T>(st + (long long)(TAPS - 1 + src) * C + c0, hist[j]);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) hist[j][e] += ib[e];
         } else {
 #pragma unroll
           for (int e = 0; e < 8; ++e) hist[j][e] = 0.f;
@@ -780,13 +877,15 @@ conv_silu_vec_kernel(const T* __restrict__ x, long long ld, const T* __restrict_
         for (int e = 0; e < 8; ++e) hist[j][e] = hist[j - 1][e];
     }
     load8_f32<T>(x + (long long)t * ld + c0, hist[0]);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) hist[0][e] += ib[e];
     float o[8];
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
       float a = b8[e];
 #pragma unroll
       for (int j = 0; j < TAPS; ++j) a += wt[e][TAPS - 1 - j] * hist[j][e];
-      o[e] = silu_f(a);
+      o[e] = act ? silu_f(a) : a;
     }
     float4* op = reinterpret_cast<float4*>(out + (long long)t * C + c0);
     op[0] = make_float4(o[0], o[1], o[2], o[3]);
@@ -874,12 +973,14 @@ __global__ void __launch_bounds__(kRecThreads)
 linear_recurrence_kernel(const float* __restrict__ kvec, const float* __restrict__ qvec, long long ldkq,
                          const float* __restrict__ val, long long ldv, const float* __restrict__ decay,
                          const float* __restrict__ beta, const float* __restrict__ skip, float* __restrict__ state,
-                         float* __restrict__ out, const int* __restrict__ seq_info, int H, int G, int n, int dv) {
+                         float* __restrict__ out, const int* __restrict__ seq_info, int H, int G, int n, int dv,
+                         int decay_ld) {
   // Lane l of a column holds the float4 chunks l, l + LPC, l + 2 LPC, ... of the column's n-vector (padded with zeros
   // to NP = LPC R), so k, q and the state move as 16-byte words without bank conflicts.  Two staging buffers, each
   // k [TB][NP] | q [TB][NP] | v [TB][COLS] | decay [TB] | beta [TB]: the next TB tokens are copied in (cp.async) while
   // the current ones are walked.  CHAN: the decay is a vector over the key channels (decay [rows, H n]) and follows the
   // scalars as one more [TB][NP] block; the state is multiplied by it chunk by chunk before the delta rule's product.
+  // decay_ld 0: the H decays are the same for every row.  beta null: every write strength is one.
   constexpr int NP = R * LPC, R4 = R / 4, COLS = kRecThreads / LPC;
   extern __shared__ __align__(16) float sm[];
   constexpr int stage = (CHAN ? 3 : 2) * kTB * NP + kTB * COLS + 2 * kTB;
@@ -889,7 +990,11 @@ linear_recurrence_kernel(const float* __restrict__ kvec, const float* __restrict
   const int lc = threadIdx.x / LPC, l = threadIdx.x % LPC;
   const int col = blockIdx.x * COLS + lc;
   const bool live = col < dv;
-  for (int i = threadIdx.x; i < 2 * stage; i += blockDim.x) sm[i] = 0.f;      // the padding stays zero
+  constexpr int beta0 = 2 * kTB * NP + kTB * COLS + kTB;
+  for (int i = threadIdx.x; i < 2 * stage; i += blockDim.x) {                 // the padding stays zero
+    const int j = i % stage - beta0;
+    sm[i] = (beta == nullptr && j >= 0 && j < kTB) ? 1.f : 0.f;
+  }
   float* sp = state + (((long long)slot * H + h) * dv + (live ? col : 0)) * n;
   const bool n4 = (n & 3) == 0;
   const bool wide_copy = n4 && (ldkq & 3) == 0 && ((reinterpret_cast<uintptr_t>(kvec) & 15) == 0) &&
@@ -958,8 +1063,8 @@ linear_recurrence_kernel(const float* __restrict__ kvec, const float* __restrict
       __pipeline_memcpy_async(sv + i, val + (long long)(first + t0 + i / COLS) * ldv + h * dv + c, 4);
     }
     for (int i = threadIdx.x; i < nt; i += blockDim.x) {
-      if (!CHAN) __pipeline_memcpy_async(sa + i, decay + (long long)(first + t0 + i) * H + h, 4);
-      __pipeline_memcpy_async(sb + i, beta + (long long)(first + t0 + i) * H + h, 4);
+      if (!CHAN) __pipeline_memcpy_async(sa + i, decay + (long long)(first + t0 + i) * decay_ld + h, 4);
+      if (beta != nullptr) __pipeline_memcpy_async(sb + i, beta + (long long)(first + t0 + i) * H + h, 4);
     }
     __pipeline_commit();
   };
@@ -1090,7 +1195,7 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 group_norm_gate_kernel(const float* __restrict__ y, const T* __restrict__ gate, long long ldg,
                        const T* __restrict__ w, int wlen, T* __restrict__ out, int C, int gs, float eps,
-                       int gate_first) {
+                       int gate_first, long long out_ld, float out_scale) {
   __shared__ float red[32];
   const int t = blockIdx.x, c0 = blockIdx.y * gs;
   const float* yr = y + (long long)t * C + c0;
@@ -1109,7 +1214,7 @@ group_norm_gate_kernel(const float* __restrict__ y, const T* __restrict__ gate, 
     const float sg = sigm ? sigmoid_f(to_f32<T>(gr[c])) : silu_f(to_f32<T>(gr[c]));
     const float wv = to_f32<T>(w[(c0 + c) % wlen]);
     const float v = gate_first ? yr[c] * sg * inv * wv : yr[c] * inv * wv * sg;
-    out[(long long)t * C + c0 + c] = from_f32<T>(v);
+    out[(long long)t * out_ld + c0 + c] = from_f32<T>(v * out_scale);
   }
 }
 
@@ -1495,18 +1600,29 @@ SXB_API int sxb_embed_sinusoid(const void* ids, const void* pos, const void* tab
   return SXB_OK;
 }
 
-/* Per row of the fp32 residual [rows, width]: if y: residual += mult * y / rms(y) * w_post (without w_post: += mult * y),
- * the addend times y_scale per channel if given; if extra (fp32): residual += extra; if w_pre: out = residual /
+/* Per row of the fp32 residual [rows, width]: if y: residual += mult * y / rms(y) * (post_add + w_post) (without w_post: +=
+ * mult * y), the addend times y_scale per channel if given; if extra (fp32): residual += extra; if w_pre: out = residual /
  * rms(residual) * (w_add + w_pre) (out without w_pre: the residual in `dtype`).  y, w_post, w_pre, y_scale, out are
  * `dtype`; any of the parts may be absent (null). */
 SXB_API int sxb_resid_norm_step(void* resid, const void* y, const void* w_post, const void* extra, const void* w_pre,
                                 void* out, long long rows, int width, float eps, float mult, int dtype,
-                                const void* y_scale, float w_add, void* stream) {
+                                const void* y_scale, float w_add, float post_add, void* stream) {
   if (rows <= 0) return SXB_OK;
   if ((y == nullptr && w_post != nullptr) || (w_pre != nullptr && out == nullptr)) return SXB_ERR_BAD_ARG;
+  if (width % 8 == 0 && width <= 8192 &&
+      ((reinterpret_cast<uintptr_t>(resid) | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(w_post) |
+        reinterpret_cast<uintptr_t>(extra) | reinterpret_cast<uintptr_t>(w_pre) | reinterpret_cast<uintptr_t>(out) |
+        reinterpret_cast<uintptr_t>(y_scale)) & 15) == 0) {
+    const int nt = (width / 8 + 31) / 32 * 32;
+    SEQMIX_DISPATCH(dtype, (resid_norm_step_vec_kernel<T><<<(unsigned)rows, nt, 0, (cudaStream_t)stream>>>(
+                               (float*)resid, (const T*)y, (const T*)w_post, (const float*)extra, (const T*)w_pre,
+                               (T*)out, width, eps, mult, (const T*)y_scale, w_add, post_add)));
+    SXB_CHECK_LAUNCH();
+    return SXB_OK;
+  }
   SEQMIX_DISPATCH(dtype, (resid_norm_step_kernel<T><<<(unsigned)rows, 256, 0, (cudaStream_t)stream>>>(
                              (float*)resid, (const T*)y, (const T*)w_post, (const float*)extra, (const T*)w_pre,
-                             (T*)out, width, eps, mult, (const T*)y_scale, w_add)));
+                             (T*)out, width, eps, mult, (const T*)y_scale, w_add, post_add)));
   SXB_CHECK_LAUNCH();
   return SXB_OK;
 }
@@ -1530,14 +1646,18 @@ SXB_API int sxb_qk_norm_append(const void* qkv, long long ld, const void* bias, 
 /* As sxb_qk_norm_append for projections that pass a short causal filter over time first (conv_w `dtype` [C, taps] with
  * C = Hq*d + G*d + G*dv, last tap = current token, or null; carried inputs state `dtype` [slots, taps-1, C], to be moved
  * on with sxb_conv_state_update afterwards), with a norm weight of d entries shared by the heads (q_w / k_w, `dtype`, or
- * null) and a query temperature 1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1). */
+ * null) and a query temperature 1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1).  Then the first n_rot channels of every
+ * q and k head turn by pos * inv_freq[i] (fp32 [n_rot / 2]) in pairs (2i, 2i+1) (interleaved != 0) or (i, i + n_rot/2), cos and
+ * sin multiplied by amp (n_rot 0: no rotation). */
 SXB_API int sxb_qkv_filter_norm_append(const void* qkv, long long ld, const void* conv_w, const void* state,
                                        const void* seq_info, const void* q_w, const void* k_w, void* q_out,
                                        void* kcache, void* vcache, const void* tok_seq, const void* tok_pos,
                                        const void* tables, int n_tokens, int max_blocks, int block_size, int Hq, int G,
                                        int d, int dv, int taps, float eps, int normalize, float temp_coef,
-                                       int temp_every, int dtype, void* stream) {
+                                       int temp_every, const void* inv_freq, int n_rot, int interleaved, float amp,
+                                       int dtype, void* stream) {
   if (n_tokens <= 0) return SXB_OK;
+  if (n_rot < 0 || n_rot > d || (n_rot & 1) || (n_rot > 0 && inv_freq == nullptr)) return SXB_ERR_BAD_ARG;
   if (d > 256 || dv > 256 || taps < 1 || taps > kMaxTaps || temp_every < 1) return SXB_ERR_UNSUPPORTED;
   if (conv_w != nullptr && taps > 1 && state == nullptr) return SXB_ERR_BAD_ARG;
   const int widest = std::max(d, dv);
@@ -1552,12 +1672,14 @@ SXB_API int sxb_qkv_filter_norm_append(const void* qkv, long long ld, const void
   const int rpw = (ktaps > 0 && n_tokens >= 1024) ? 8 : 1;
   const dim3 grid((n_tokens + rpw - 1) / rpw, (Hq + 2 * G + 3) / 4);
   if (conv_w == nullptr) taps = 1;
+  const size_t smem = n_rot > 0 ? (size_t)(rpw * n_rot + 4 * 32 * vecw) * sizeof(float) : 0;
 #define FILTER_APPEND_T(VEC, TAPS)                                                                                     \
-  SEQMIX_DISPATCH(dtype, (qkv_filter_norm_append_kernel<T, VEC, TAPS><<<grid, 128, 0, (cudaStream_t)stream>>>(         \
+  SEQMIX_DISPATCH(dtype, (qkv_filter_norm_append_kernel<T, VEC, TAPS><<<grid, 128, smem, (cudaStream_t)stream>>>(      \
                              (const T*)qkv, ld, (const T*)conv_w, (const T*)state, (const int*)seq_info, (const T*)q_w, \
                              (const T*)k_w, (float*)q_out, (T*)kcache, (T*)vcache, (const int*)tok_seq,                \
                              (const int*)tok_pos, (const int*)tables, max_blocks, block_size, Hq, G, d, dv, taps, eps, \
-                             normalize, temp_coef, temp_every, vec_ok, n_tokens, rpw)))
+                             normalize, temp_coef, temp_every, vec_ok, n_tokens, rpw, (const float*)inv_freq, n_rot,   \
+                             interleaved, amp)))
 #define FILTER_APPEND(VEC)                 \
   do {                                     \
     if (ktaps == 2) FILTER_APPEND_T(VEC, 2);      \
@@ -1582,19 +1704,22 @@ SXB_API int sxb_qkv_filter_norm_append(const void* qkv, long long ld, const void
  * column range of the key rows.  out `dtype` [n_tokens, Hq * dv] (the caches have the same type).  dist_bias (fp32
  * [Hq, bias_len] or null) is added to the scaled score of a key at distance n = query position - key position:
  * dist_bias[h, min(n, bias_len - 1)].  gate (`dtype` rows of pitch gate_ld with Hq * dv channels, or Hq when
- * gate_heads != 0, or null): the output is multiplied by sigmoid(gate), per channel or per head.  One CTA per (token, head group). */
+ * gate_heads != 0, or null): the output is multiplied by sigmoid(gate), per channel or per head.  Output rows have pitch
+ * out_ld (0 = Hq * dv) and are multiplied by out_scale.  One CTA per (token, head group). */
 SXB_API int sxb_sink_attention(const void* q, const void* kcache, const void* vcache, const void* sink, void* out,
                                const void* tok_seq, const void* tok_pos, const void* tables, int n_tokens,
                                int max_blocks, int block_size, int Hq, int G, int d, int dv, float scale, int chunk,
                                int window, int k_pitch, int v_pitch, const void* dist_bias, int bias_len,
-                               const void* gate, long long gate_ld, int gate_heads, int dtype, void* stream) {
+                               const void* gate, long long gate_ld, int gate_heads, long long out_ld, float out_scale, int dtype,
+                               void* stream) {
   if (n_tokens <= 0) return SXB_OK;
   if (dv > 32 * kMaxVPerLane || Hq % G || (dist_bias != nullptr && bias_len < 1)) return SXB_ERR_UNSUPPORTED;
   if (k_pitch <= 0) k_pitch = G * d;
   if (v_pitch <= 0) v_pitch = G * dv;
+  if (out_ld <= 0) out_ld = (long long)Hq * dv;
   const int rc = attention_rows(dtype, dim3(n_tokens, 1), q, kcache, vcache, sink, out, tok_seq, tok_pos, tables,
                                 max_blocks, block_size, Hq, G, d, dv, scale, chunk, window, k_pitch, v_pitch, nullptr,
-                                dist_bias, bias_len, gate, gate_ld, gate_heads, (cudaStream_t)stream);
+                                dist_bias, bias_len, gate, gate_ld, gate_heads, out_ld, out_scale, (cudaStream_t)stream);
   if (rc != SXB_OK) return rc;
   SXB_CHECK_LAUNCH();
   return SXB_OK;
@@ -1715,7 +1840,8 @@ static int launch_attention_tiles(const void* q, const void* kcache, const void*
                                   const void* atoms, int n_long, const void* tables, int max_blocks, int block_size,
                                   int Hq, int G, int d, int dv, float scale, int chunk, int window, int kpitch,
                                   int vpitch, const void* dist_bias, int bias_len, const void* gate,
-                                  long long gate_ld, int gate_heads, cudaStream_t s) {
+                                  long long gate_ld, int gate_heads, long long out_ld,
+                                   float out_scale, cudaStream_t s) {
   const size_t smem = (size_t)(kBQ * (d + 4) + std::max(kBK * (d + 4), kBQ * (kBK + 4)) + kBK * NV * 64) * sizeof(float);
   cudaError_t e = cudaFuncSetAttribute(sink_attention_tile_kernel<T, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                        (int)smem);
@@ -1723,7 +1849,7 @@ static int launch_attention_tiles(const void* q, const void* kcache, const void*
   sink_attention_tile_kernel<T, NV><<<dim3(2 * n_long, Hq), 256, smem, s>>>(
       (const float*)q, (const T*)kcache, (const T*)vcache, (const float*)sink, (T*)out, (const int*)atoms,
       (const int*)tables, max_blocks, block_size, Hq, G, d, dv, scale, chunk, window, kpitch, vpitch,
-      (const float*)dist_bias, bias_len, (const T*)gate, gate_ld, gate_heads);
+      (const float*)dist_bias, bias_len, (const T*)gate, gate_ld, gate_heads, out_ld, out_scale);
   return SXB_OK;
 }
 
@@ -1734,11 +1860,13 @@ SXB_API int sxb_sink_attention_atoms(const void* q, const void* kcache, const vo
                                      const void* atoms, int n_atoms, int n_long, const void* tables, int max_blocks,
                                      int block_size, int Hq, int G, int d, int dv, float scale, int chunk, int window,
                                      int k_pitch, int v_pitch, const void* dist_bias, int bias_len, const void* gate,
-                                     long long gate_ld, int gate_heads, int dtype, void* stream) {
+                                     long long gate_ld, int gate_heads, long long out_ld, float out_scale, int dtype,
+                               void* stream) {
   if (n_atoms <= 0) return SXB_OK;
   if (dist_bias != nullptr && bias_len < 1) return SXB_ERR_UNSUPPORTED;
   if (k_pitch <= 0) k_pitch = G * d;
   if (v_pitch <= 0) v_pitch = G * dv;
+  if (out_ld <= 0) out_ld = (long long)Hq * dv;
   if (d % 4 || dv % 4 || k_pitch % 4 || v_pitch % 4 || d > 256 || dv > 256 || Hq % G || n_long < 0 || n_long > n_atoms)
     return SXB_ERR_UNSUPPORTED;
   cudaStream_t s = (cudaStream_t)stream;
@@ -1749,7 +1877,7 @@ SXB_API int sxb_sink_attention_atoms(const void* q, const void* kcache, const vo
   SEQMIX_DISPATCH(dtype, (rc = launch_attention_tiles<T, NV>(q, kcache, vcache, sink, out, atoms, n_long, tables,      \
                                                               max_blocks, block_size, Hq, G, d, dv, scale, chunk,      \
                                                               window, k_pitch, v_pitch, dist_bias, bias_len, gate,     \
-                                                              gate_ld, gate_heads, s)))
+                                                              gate_ld, gate_heads, out_ld, out_scale, s)))
     if (nv == 1) TILES(1);
     else if (nv == 2) TILES(2);
     else if (nv == 3) TILES(3);
@@ -1761,19 +1889,19 @@ SXB_API int sxb_sink_attention_atoms(const void* q, const void* kcache, const vo
   if (n_atoms > n_long) {
     const int rc = attention_rows(dtype, dim3((n_atoms - n_long) * kShortAtom, 1), q, kcache, vcache, sink, out, nullptr,
                                   nullptr, tables, max_blocks, block_size, Hq, G, d, dv, scale, chunk, window, k_pitch,
-                                  v_pitch, (const int*)atoms + 6 * n_long, dist_bias, bias_len, gate, gate_ld, gate_heads, s);
+                                  v_pitch, (const int*)atoms + 6 * n_long, dist_bias, bias_len, gate, gate_ld, gate_heads, out_ld, out_scale, s);
     if (rc != SXB_OK) return rc;
     SXB_CHECK_LAUNCH();
   }
   return SXB_OK;
 }
 
-/* Short causal filter + SiLU over C channels of x [n_tokens, ld] (`dtype`), w [C, taps] (last tap = current token),
- * bias [C] or null, carried inputs state [slots, taps-1, C]; out fp32 [n_tokens, C].  seq_info int32 [n_seqs, 4] =
+/* Short causal filter + SiLU (act 1; act 0: no activation) over C channels of x [n_tokens, ld] (`dtype`), w [C, taps] (last
+ * tap = current token), in_bias [C] added to every input row of the sequence (or null), bias [C] added to the sum (or null), carried inputs state [slots, taps-1, C]; out fp32 [n_tokens, C].  seq_info int32 [n_seqs, 4] =
  * {first row, rows, seen tokens, slot}. */
 SXB_API int sxb_conv_silu(const void* x, long long ld, const void* w, const void* bias, const void* state,
                           const void* seq_info, const void* tok_seq, void* out, int n_tokens, int C, int taps,
-                          int dtype, void* stream) {
+                          const void* in_bias, int act, int dtype, void* stream) {
   if (n_tokens <= 0) return SXB_OK;
   if (taps < 1 || taps > kMaxTaps) return SXB_ERR_UNSUPPORTED;
   const bool aligned = ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(state) |
@@ -1784,7 +1912,7 @@ SXB_API int sxb_conv_silu(const void* x, long long ld, const void* w, const void
 #define CONV_VEC(TAPS)                                                                                             \
   SEQMIX_DISPATCH(dtype, (conv_silu_vec_kernel<T, TAPS><<<vgrid, 128, 0, (cudaStream_t)stream>>>(                  \
                              (const T*)x, ld, (const T*)w, (const T*)bias, (const T*)state, (const int*)seq_info,  \
-                             (const int*)tok_seq, (float*)out, C, n_tokens)))
+                             (const int*)tok_seq, (float*)out, C, n_tokens, (const T*)in_bias, act)))
     if (taps == 2) CONV_VEC(2);
     else if (taps == 3) CONV_VEC(3);
     else CONV_VEC(4);
@@ -1795,7 +1923,7 @@ SXB_API int sxb_conv_silu(const void* x, long long ld, const void* w, const void
   dim3 grid(n_tokens, (C + 1023) / 1024);
   SEQMIX_DISPATCH(dtype, (conv_silu_kernel<T><<<grid, 256, 0, (cudaStream_t)stream>>>(
                              (const T*)x, ld, (const T*)w, (const T*)bias, (const T*)state, (const int*)seq_info,
-                             (const int*)tok_seq, (float*)out, C, taps)));
+                             (const int*)tok_seq, (float*)out, C, taps, (const T*)in_bias, act)));
   SXB_CHECK_LAUNCH();
   return SXB_OK;
 }
@@ -1841,14 +1969,15 @@ SXB_API int sxb_recurrence_gates(const void* a_raw, const void* b_raw, long long
 /* decay_channels != 0: decay fp32 [rows, H * n] holds one factor per (head, key channel) pair (it scales the state entries of that key channel).
  * Per sequence and head, rows in order:  S <- decay S;  u = beta (v - [delta] S^T k);  S <- S + k u^T;
  * o = S^T q (+ skip[h] v).  kvec / qvec fp32 [rows, ldkq] hold G heads of n channels, val fp32 [rows, ldv] H heads of dv,
- * decay / beta fp32 [rows, H], state fp32 [slots, H, dv, n] (taken as zero when the sequence has seen no token), out fp32
+ * decay / beta fp32 [rows, H] (fixed_decay != 0: decay fp32 [H], the same for every row; beta null: ones), state fp32 [slots, H, dv, n] (taken as zero when the sequence has seen no token), out fp32
  * [rows, H * dv]. */
 SXB_API int sxb_linear_recurrence(const void* kvec, const void* qvec, long long ldkq, const void* val, long long ldv,
                                   const void* decay, const void* beta, const void* skip, void* state, void* out,
                                   const void* seq_info, int n_seqs, int H, int G, int n, int dv, int delta,
-                                  int decay_channels, void* stream) {
+                                  int decay_channels, int fixed_decay, void* stream) {
   if (n_seqs <= 0) return SXB_OK;
   if (n > 256 || H % G) return SXB_ERR_UNSUPPORTED;
+  if (decay_channels && fixed_decay) return SXB_ERR_BAD_ARG;
   cudaStream_t s = (cudaStream_t)stream;
 #define LAUNCH_REC(R, D, LPC, CH)                                                                                   \
   do {                                                                                                              \
@@ -1859,7 +1988,8 @@ SXB_API int sxb_linear_recurrence(const void* kvec, const void* qvec, long long 
                            (int)smem);                                                                              \
     linear_recurrence_kernel<R, D, LPC, CH><<<dim3((dv + cols - 1) / cols, H, n_seqs), kRecThreads, smem, s>>>(     \
         (const float*)kvec, (const float*)qvec, ldkq, (const float*)val, ldv, (const float*)decay,                  \
-        (const float*)beta, (const float*)skip, (float*)state, (float*)out, (const int*)seq_info, H, G, n, dv);     \
+        (const float*)beta, (const float*)skip, (float*)state, (float*)out, (const int*)seq_info, H, G, n, dv,      \
+        fixed_decay ? 0 : H);                                                                                       \
   } while (0)
 #define LAUNCH_REC_N(D, CH)                                  \
   if (n <= 32) LAUNCH_REC(4, D, 8, CH);                      \
@@ -1879,14 +2009,17 @@ SXB_API int sxb_linear_recurrence(const void* kvec, const void* qvec, long long 
 
 /* RMS norm over groups of gs channels of y fp32 [n_tokens, C] with a SiLU gate (`dtype` rows of pitch ldg) and a weight
  * of wlen entries that repeats along the row.  gate_first bit 0: norm(y silu(gate)) w; else norm(y) w silu(gate); bit 1:
- * sigmoid(gate) in place of silu(gate). */
+ * sigmoid(gate) in place of silu(gate).  Output rows have pitch out_ld (0 = C) and are multiplied by out_scale. */
 SXB_API int sxb_group_norm_gate(const void* y, const void* gate, long long ldg, const void* w, int wlen, void* out,
-                                int n_tokens, int C, int gs, float eps, int gate_first, int dtype, void* stream) {
+                                int n_tokens, int C, int gs, float eps, int gate_first, long long out_ld,
+                                float out_scale, int dtype, void* stream) {
   if (n_tokens <= 0) return SXB_OK;
   if (gs <= 0 || C % gs) return SXB_ERR_BAD_ARG;
+  if (out_ld <= 0) out_ld = C;
   dim3 grid(n_tokens, C / gs);
   SEQMIX_DISPATCH(dtype, (group_norm_gate_kernel<T><<<grid, 128, 0, (cudaStream_t)stream>>>(
-                             (const float*)y, (const T*)gate, ldg, (const T*)w, wlen, (T*)out, C, gs, eps, gate_first)));
+                             (const float*)y, (const T*)gate, ldg, (const T*)w, wlen, (T*)out, C, gs, eps, gate_first,
+                             out_ld, out_scale)));
   SXB_CHECK_LAUNCH();
   return SXB_OK;
 }

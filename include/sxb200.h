@@ -451,7 +451,7 @@ int sxb_embed_sinusoid(const void* ids, const void* pos, const void* table, void
                        float scale, float base, int dtype, void* stream);
 int sxb_resid_norm_step(void* resid, const void* y, const void* w_post, const void* extra, const void* w_pre,
                         void* out, long long rows, int width, float eps, float mult, int dtype,
-                        const void* y_scale, float w_add, void* stream);
+                        const void* y_scale, float w_add, float post_add, void* stream);
 int sxb_qk_norm_append(const void* qkv, long long ld, const void* bias, void* q_out, void* kcache, void* vcache,
                        const void* tok_seq, const void* tok_pos, const void* tables, int n_tokens, int max_blocks,
                        int block_size, int Hq, int G, int d, int dv, float eps, int normalize, int dtype,
@@ -460,10 +460,11 @@ int sxb_sink_attention(const void* q, const void* kcache, const void* vcache, co
                        const void* tok_seq, const void* tok_pos, const void* tables, int n_tokens, int max_blocks,
                        int block_size, int Hq, int G, int d, int dv, float scale, int chunk, int window,
                        int k_pitch, int v_pitch, const void* dist_bias, int bias_len, const void* gate,
-                       long long gate_ld, int gate_heads, int dtype, void* stream);
+                       long long gate_ld, int gate_heads, long long out_ld, float out_scale, int dtype,
+                       void* stream);
 int sxb_conv_silu(const void* x, long long ld, const void* w, const void* bias, const void* state,
-                  const void* seq_info, const void* tok_seq, void* out, int n_tokens, int C, int taps, int dtype,
-                  void* stream);
+                  const void* seq_info, const void* tok_seq, void* out, int n_tokens, int C, int taps,
+                  const void* in_bias, int act, int dtype, void* stream);
 int sxb_conv_state_update(const void* x, long long ld, void* state, const void* seq_info, int n_seqs, int C,
                           int taps, int dtype, void* stream);
 int sxb_unit_norm_heads(void* x, long long ld, int col0, int n_heads, int dim, float mult, float eps, int n_tokens,
@@ -474,9 +475,10 @@ int sxb_recurrence_gates(const void* a_raw, const void* b_raw, long long ld, con
 int sxb_linear_recurrence(const void* kvec, const void* qvec, long long ldkq, const void* val, long long ldv,
                           const void* decay, const void* beta, const void* skip, void* state, void* out,
                           const void* seq_info, int n_seqs, int H, int G, int n, int dv, int delta,
-                          int decay_channels, void* stream);
+                          int decay_channels, int fixed_decay, void* stream);
 int sxb_group_norm_gate(const void* y, const void* gate, long long ldg, const void* w, int wlen, void* out,
-                        int n_tokens, int C, int gs, float eps, int gate_first, int dtype, void* stream);
+                        int n_tokens, int C, int gs, float eps, int gate_first, long long out_ld, float out_scale,
+                        int dtype, void* stream);
 int sxb_gated_act_rows(const void* in, void* out, long long rows, int F, int act, int dtype, float limit,
                        void* stream);
 
@@ -485,7 +487,8 @@ int sxb_sink_attention_atoms(const void* q, const void* kcache, const void* vcac
                              const void* atoms, int n_atoms, int n_long, const void* tables, int max_blocks,
                              int block_size, int Hq, int G, int d, int dv, float scale, int chunk, int window,
                              int k_pitch, int v_pitch, const void* dist_bias, int bias_len, const void* gate,
-                             long long gate_ld, int gate_heads, int dtype, void* stream);
+                             long long gate_ld, int gate_heads, long long out_ld, float out_scale, int dtype,
+                             void* stream);
 
 /* ---- csrc/moe_ragged.cu */
 /* As sxb_moe_scatter with every copied row multiplied by its routing weight: moe_input[slot(t, k)] = x[t] * scores[t, k].
@@ -524,7 +527,8 @@ int sxb_qkv_filter_norm_append(const void* qkv, long long ld, const void* conv_w
                                const void* seq_info, const void* q_w, const void* k_w, void* q_out, void* kcache,
                                void* vcache, const void* tok_seq, const void* tok_pos, const void* tables,
                                int n_tokens, int max_blocks, int block_size, int Hq, int G, int d, int dv,
-                               int taps, float eps, int normalize, float temp_coef, int temp_every, int dtype,
+                               int taps, float eps, int normalize, float temp_coef, int temp_every,
+                               const void* inv_freq, int n_rot, int interleaved, float amp, int dtype,
                                void* stream);
 int sxb_side_gate(const void* gx, long long ld, const void* table, long long table_ld, const void* ids, void* out,
                   int n_tokens, int dim, int out_w, int col0, int dtype, void* stream);
@@ -540,10 +544,12 @@ int sxb_router_logits(const void* x, long long ld, const void* w, const void* bi
 /* Group-limited gating with a choice correction.  logits fp32 [T, E]; correction fp32 [E] or null; the E experts form
  * n_groups contiguous blocks of equal size of which the keep_groups whose best (score + correction) is largest stay eligible;
  * the top_k largest (score + correction) among them win; scores fp32 [T, K] = softmax score of the winner / (sum of the
- * winners' scores + 1e-20) * scale; assignments / offsets / expert_counts as sxb_top_k_gating. */
+ * winners' scores + 1e-20) * scale; assignments / offsets / expert_counts as sxb_top_k_gating.  flags: 1 = the score is the
+ * sigmoid of the expert's own logit, 2 = groups are ranked by the sum of their two largest (score + correction), 4 = the
+ * winners' scores are not divided by their sum. */
 int sxb_grouped_top_k_gating(const void* logits, const void* correction, void* scores, void* assignments,
                              void* offsets, void* expert_counts, int n_tokens, int n_experts, int top_k,
-                             int n_groups, int keep_groups, float scale, void* stream);
+                             int n_groups, int keep_groups, float scale, int flags, void* stream);
 /* dst rows [offsets[g_lo], offsets[g_hi]) <- src rows of the same range; rows of row_bytes (a multiple of 16) bytes,
  * offsets int32 on the device (group row offsets of an expert-sorted buffer), max_rows bounds the grid. */
 int sxb_copy_group_rows(const void* src, void* dst, const void* offsets, int g_lo, int g_hi, int row_bytes,
@@ -569,13 +575,24 @@ int sxb_norm_filter_rows(const void* x, const void* rstd, const void* w1, const 
 int sxb_rope_append(const void* proj, long long ld, int q0, int k0, int v0, const void* q_w, const void* k_w,
                     const void* inv_freq, const void* q_scale, void* q_out, void* kcache, void* vcache,
                     const void* tok_seq, const void* tok_pos, const void* tables, int n_tokens, int max_blocks,
-                    int block_size, int Hq, int G, int d, int dv, int n_rot, int interleaved, float eps, int dtype,
-                    void* stream);
+                    int block_size, int Hq, int G, int d, int dv, int n_rot, int interleaved, float eps, float amp,
+                    int dtype, void* stream);
 int sxb_removal_prepare(const void* proj, long long ld, int r0, int k0, int v0, int a0, int low0, const void* w2,
                         const void* w0, const void* a_bias, void* buf, int n_tokens, int H, int n, int rank,
                         float rate, float eps, int dtype, void* stream);
 int sxb_removal_recurrence(const void* buf, void* state, void* out, const void* seq_info, int n_seqs, int H, int n,
                            int single_rows, void* stream);
+
+/* ---- csrc/gated_mixers.cu */
+int sxb_silu_columns(const void* x, long long ld, void* out, int n_tokens, int C, int dtype, void* stream);
+int sxb_decay_prepare(const void* proj, long long ld, int q0, int k0, int v0, int low0, const void* w2,
+                      const void* bias, void* buf, void* decay, int n_tokens, int Hn, int Hv, int rank,
+                      float qscale, float inv_tau, int dtype, void* stream);
+int sxb_lru_gates(const void* u, const void* w, const void* bias, const void* rate, void* a_out, void* g_out,
+                  int n_tokens, int N, int blocks, int dtype, void* stream);
+int sxb_lru_scan(const void* a, const void* g, const void* y, long long ldy, const void* ybias, const void* x,
+                 long long ldx, void* state, void* conv_state, const void* seq_info, void* out, long long out_ld,
+                 int n_seqs, int N, int keep, float scale, int single_rows, int dtype, void* stream);
 
 #ifdef __cplusplus
 }

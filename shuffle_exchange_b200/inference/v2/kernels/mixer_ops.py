@@ -18,17 +18,17 @@ from ....native import lib as _lib
 
 _lib.register({
     "sxb_embed_sinusoid": "pppp" "ii" "ff" "i" "p",
-    "sxb_resid_norm_step": "pppppp" "l" "i" "ff" "i" "p" "f" "p",
+    "sxb_resid_norm_step": "pppppp" "l" "i" "ff" "i" "p" "ff" "p",
     "sxb_qk_norm_append": "p" "l" "ppppppp" "iiiiiii" "f" "ii" "p",
-    "sxb_qkv_filter_norm_append": "p" "l" "ppppppppppp" "iiiiiiii" "f" "i" "f" "i" "i" "p",
-    "sxb_sink_attention": "pppppppp" "iiiiiii" "f" "iiii" "p" "i" "p" "l" "ii" "p",
-    "sxb_sink_attention_atoms": "pppppp" "ii" "p" "iiiiii" "f" "iiii" "p" "i" "p" "l" "ii" "p",
-    "sxb_conv_silu": "p" "l" "pppppp" "iii" "i" "p",
+    "sxb_qkv_filter_norm_append": "p" "l" "ppppppppppp" "iiiiiiii" "f" "i" "f" "i" "p" "ii" "f" "i" "p",
+    "sxb_sink_attention": "pppppppp" "iiiiiii" "f" "iiii" "p" "i" "p" "l" "i" "l" "f" "i" "p",
+    "sxb_sink_attention_atoms": "pppppp" "ii" "p" "iiiiii" "f" "iiii" "p" "i" "p" "l" "i" "l" "f" "i" "p",
+    "sxb_conv_silu": "p" "l" "pppppp" "iii" "p" "i" "i" "p",
     "sxb_conv_state_update": "p" "l" "pp" "iii" "i" "p",
     "sxb_unit_norm_heads": "p" "l" "iii" "ff" "i" "p",
     "sxb_recurrence_gates": "pp" "l" "pppp" "iii" "i" "p",
-    "sxb_linear_recurrence": "pp" "l" "p" "l" "pppppp" "iiiiii" "i" "p",
-    "sxb_group_norm_gate": "pp" "l" "p" "i" "p" "iii" "f" "i" "i" "p",
+    "sxb_linear_recurrence": "pp" "l" "p" "l" "pppppp" "iiiiii" "ii" "p",
+    "sxb_group_norm_gate": "pp" "l" "p" "i" "p" "iii" "f" "i" "l" "f" "i" "p",
     "sxb_gated_act_rows": "pp" "l" "ii" "i" "f" "p",
     "sxb_conv_residual": "pppppp" "iii" "i" "p",
     "sxb_post_norm_mix": "pppppp" "l" "i" "pp" "l" "i" "f" "i" "p",
@@ -62,6 +62,15 @@ def _rows(t: torch.Tensor) -> torch.Tensor:
     return t
 
 
+def _out_rows(out: Optional[torch.Tensor], T: int, width: int, dtype: torch.dtype, device) -> torch.Tensor:
+    """The caller's output rows (checked), or new ones."""
+    if out is None:
+        return torch.empty(T, width, dtype=dtype, device=device)
+    if tuple(out.shape) != (T, width) or out.dtype != dtype:
+        raise ValueError(f"expected output rows [{T}, {width}] of {dtype}, got {tuple(out.shape)} of {out.dtype}")
+    return _rows(out)
+
+
 # ------------------------------------------------------------------------------------------------ embedding
 def embed_sinusoid(ids: torch.Tensor, positions: torch.Tensor, table: torch.Tensor, scale: float,
                    base: Optional[float] = 10000.0) -> torch.Tensor:
@@ -90,11 +99,13 @@ def _rms(x: torch.Tensor, eps: float) -> torch.Tensor:
 def resid_norm_step(resid: torch.Tensor, y: Optional[torch.Tensor], w_post: Optional[torch.Tensor],
                     extra: Optional[torch.Tensor], w_pre: Optional[torch.Tensor], eps: float,
                     out_dtype: torch.dtype, mult: float = 1.0, copy_out: bool = False,
-                    y_scale: Optional[torch.Tensor] = None, w_add: float = 0.0) -> Optional[torch.Tensor]:
-    """In place on the fp32 residual ``[T, W]``: ``+= mult * rms_norm(y) * w_post`` (if ``y``; without ``w_post``:
-    ``+= mult * y``; with ``y_scale`` ``[W]`` the addend is also scaled per channel), ``+= extra`` (if given); returns
-    ``rms_norm(residual) * (w_add + w_pre)`` in ``out_dtype`` (``w_add = 1`` for weights stored as their distance from
-    one; without ``w_pre``: the residual itself in ``out_dtype`` if ``copy_out``, else None).  One pass per row."""
+                    y_scale: Optional[torch.Tensor] = None, w_add: float = 0.0,
+                    post_add: float = 0.0) -> Optional[torch.Tensor]:
+    """In place on the fp32 residual ``[T, W]``: ``+= mult * rms_norm(y) * (post_add + w_post)`` (if ``y``; without
+    ``w_post``: ``+= mult * y``; with ``y_scale`` ``[W]`` the addend is also scaled per channel), ``+= extra`` (if given);
+    returns ``rms_norm(residual) * (w_add + w_pre)`` in ``out_dtype`` (``w_add``, ``post_add`` 1 for weights stored as their
+    distance from one; without ``w_pre``: the residual itself in ``out_dtype`` if ``copy_out``, else None).  One pass per
+    row."""
     T, W = resid.shape
     if resid.is_cuda:
         out = torch.empty(T, W, dtype=out_dtype, device=resid.device) if (w_pre is not None or copy_out) else None
@@ -103,10 +114,10 @@ def resid_norm_step(resid: torch.Tensor, y: Optional[torch.Tensor], w_post: Opti
             raise ValueError("the channel scale is stored in the activation dtype")
         _lib.call("sxb_resid_norm_step", resid.data_ptr(), _lib.ptr(y), _lib.ptr(w_post), _lib.ptr(extra),
                   _lib.ptr(w_pre), _lib.ptr(out), T, W, float(eps), float(mult), code, _lib.ptr(y_scale), float(w_add),
-                  _lib.stream_ptr())
+                  float(post_add), _lib.stream_ptr())
         return out
     if y is not None:
-        add = mult * (_rms(y.float(), eps) * w_post.float() if w_post is not None else y.float())
+        add = mult * (_rms(y.float(), eps) * (post_add + w_post.float()) if w_post is not None else y.float())
         resid += add * y_scale.float() if y_scale is not None else add
     if extra is not None:
         resid += extra
@@ -143,28 +154,49 @@ def qk_norm_append(qkv: torch.Tensor, bias: Optional[torch.Tensor], kcache: torc
     return q.contiguous()
 
 
+def rotate_heads(x: torch.Tensor, pos: torch.Tensor, inv_freq: torch.Tensor, interleaved: bool, amp: float = 1.0) -> torch.Tensor:
+    """Heads ``x`` fp32 ``[T, H, d]``: the pairs ``(2i, 2i+1)`` if ``interleaved``, else ``(i, i + len(inv_freq))``, turn by
+    ``pos * inv_freq[i]``, cos and sin times ``amp``; the channels behind them pass."""
+    half = inv_freq.numel()
+    ang = pos.float()[:, None, None] * inv_freq.float()
+    c, s = ang.cos() * amp, ang.sin() * amp
+    out = x.clone()
+    if interleaved:
+        u, v = x[..., 0: 2 * half: 2], x[..., 1: 2 * half: 2]
+        out[..., 0: 2 * half: 2], out[..., 1: 2 * half: 2] = u * c - v * s, v * c + u * s
+    else:
+        u, v = x[..., :half], x[..., half: 2 * half]
+        out[..., :half], out[..., half: 2 * half] = u * c - v * s, v * c + u * s
+    return out
+
+
 def qkv_filter_norm_append(qkv: torch.Tensor, conv_w: Optional[torch.Tensor], state: Optional[torch.Tensor],
                            seq_info: torch.Tensor, q_w: Optional[torch.Tensor], k_w: Optional[torch.Tensor],
                            kcache: torch.Tensor, vcache: torch.Tensor, tok_seq: torch.Tensor, tok_pos: torch.Tensor,
                            tables: torch.Tensor, Hq: int, G: int, d: int, dv: int, eps: float, normalize: bool = True,
-                           temp_coef: float = 0.0, temp_every: int = 1) -> torch.Tensor:
+                           temp_coef: float = 0.0, temp_every: int = 1, inv_freq: Optional[torch.Tensor] = None,
+                           interleaved: bool = False, amp: float = 1.0) -> torch.Tensor:
     """:func:`qk_norm_append` for projections ``qkv`` ``[T, >= Hq*d + G*d + G*dv]`` that first pass a short causal filter
     over time on every channel (``conv_w`` ``[C, taps]``, last column = current token; inputs before this batch's rows
     from ``state`` ``[slots, taps-1, C]``, before the sequence's start zero; None: no filter -- call
     :func:`conv_state_update` on the same columns afterwards).  q and k heads are then divided by their root mean square
     (``normalize``) and multiplied by ``q_w`` / ``k_w`` (``[d]``, shared by the heads; None: no weight); q also by
-    ``1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1)``.  Returns q fp32 ``[T, Hq, d]``; k, v go to the caches."""
+    ``1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1)``.  With ``inv_freq`` (fp32) the first ``2 len(inv_freq)`` channels of
+    every q and k head then turn by ``pos * inv_freq[i]`` (see :func:`rotate_heads`).  Returns q fp32 ``[T, Hq, d]``; k, v go
+    to the caches."""
     T = qkv.shape[0]
     bs = kcache.shape[1]
     C = (Hq + G) * d + G * dv
     taps = conv_w.shape[1] if conv_w is not None else 1
+    n_rot = 0 if inv_freq is None else 2 * inv_freq.numel()
     if qkv.is_cuda:
         q = torch.empty(T, Hq, d, dtype=torch.float32, device=qkv.device)
         _lib.call("sxb_qkv_filter_norm_append", _rows(qkv).data_ptr(), qkv.stride(0), _lib.ptr(conv_w),
                   _lib.ptr(state if taps > 1 else None), seq_info.data_ptr(), _lib.ptr(q_w), _lib.ptr(k_w),
                   q.data_ptr(), kcache.data_ptr(), vcache.data_ptr(), tok_seq.data_ptr(), tok_pos.data_ptr(),
                   tables.data_ptr(), T, tables.shape[1], bs, Hq, G, d, dv, taps, float(eps), int(normalize),
-                  float(temp_coef), int(temp_every), _dt(qkv), _lib.stream_ptr())
+                  float(temp_coef), int(temp_every), inv_freq.data_ptr() if n_rot else None, n_rot, int(interleaved),
+                  float(amp), _dt(qkv), _lib.stream_ptr())
         return q
     x = qkv[:, :C].float()
     if conv_w is not None:
@@ -193,6 +225,8 @@ def qkv_filter_norm_append(qkv: torch.Tensor, conv_w: Optional[torch.Tensor], st
     if temp_coef != 0.0:
         steps = torch.div(tok_pos.long() + 1, int(temp_every), rounding_mode="floor") + 1
         q = q * (1.0 + temp_coef * torch.log(steps.float()))[:, None, None]
+    if n_rot:
+        q, k = (rotate_heads(z, tok_pos, inv_freq, interleaved, amp) for z in (q, k))
     page = tables[tok_seq.long(), (tok_pos // bs).long()].long()
     off = (tok_pos % bs).long()
     kcache[page, off] = k.to(kcache.dtype)
@@ -211,7 +245,8 @@ def sink_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, 
                    tok_seq: torch.Tensor, tok_pos: torch.Tensor, tables: torch.Tensor, scale: float, chunk: int,
                    out_dtype: torch.dtype, atoms: Optional[torch.Tensor] = None, n_long: int = 0, window: int = 0,
                    value_cols: int = 0, value_col0: int = 0, dist_bias: Optional[torch.Tensor] = None,
-                   gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   gate: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
+                   out_scale: float = 1.0) -> torch.Tensor:
     """Softmax attention of each token (fp32 ``q`` ``[T, Hq, d]``) over the cached keys ``lo..pos`` of its sequence,
     ``lo`` = first position of the token's chunk of ``chunk`` positions, or ``pos - window + 1`` (not below 0) for a
     sliding ``window``, or 0 (both 0: plain causal).  ``sink`` (fp32 ``[Hq]``) adds ``exp(sink[h])`` to the
@@ -223,7 +258,8 @@ def sink_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, 
 
     ``dist_bias`` (fp32 ``[Hq, L]``): ``dist_bias[h, min(pos - j, L - 1)]`` is added to the scaled score of key ``j``.
     ``gate`` (``[T, Hq * dv]``, or ``[T, Hq]`` for one per head; a column slice is fine): the result is multiplied by
-    ``sigmoid(gate)``.
+    ``sigmoid(gate)``.  ``out`` (rows of ``Hq * dv`` columns, a column slice is fine) receives the result, multiplied by
+    ``out_scale`` before it is rounded.
 
     With the batch's attention ``atoms`` (longest first) of which the first ``n_long`` hold more than
     :data:`SHORT_ATOM` queries, those run the tiled kernel (64 queries per CTA, K/V tiles shared by them) and the rest
@@ -239,7 +275,7 @@ def sink_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, 
     if q.is_cuda:
         if kcache.dtype != out_dtype or vsrc.dtype != out_dtype:
             raise ValueError("the caches and the output share one activation dtype")
-        out = torch.empty(T, Hq * dv, dtype=out_dtype, device=q.device)
+        out = _out_rows(out, T, Hq * dv, out_dtype, q.device)
         vptr = vsrc.data_ptr() + (value_col0 * vsrc.element_size() if value_cols > 0 else 0)
         if value_cols > 0 and value_col0 % 8:
             raise ValueError("value columns start at a multiple of 8")
@@ -252,7 +288,7 @@ def sink_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, 
             raise ValueError("the gate has one column per head or per output channel")
         extra = (_lib.ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[1],
                  None if gate is None else _rows(gate).data_ptr(), 0 if gate is None else gate.stride(0),
-                 int(gate is not None and gate.shape[1] == Hq))
+                 int(gate is not None and gate.shape[1] == Hq), out.stride(0), float(out_scale))
         if atoms is not None and n_long > 0 and tiles_supported(d, dv):
             _lib.call("sxb_sink_attention_atoms", q.data_ptr(), kcache.data_ptr(), vptr, _lib.ptr(sink),
                       out.data_ptr(), atoms.data_ptr(), atoms.shape[0], int(n_long), tables.data_ptr(), tables.shape[1],
@@ -264,7 +300,7 @@ def sink_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, 
                   G, d, dv, float(scale), int(chunk), int(window), 0, v_pitch, *extra, _lib.dtype_code(out_dtype),
                   _lib.stream_ptr())
         return out
-    out = torch.empty(T, Hq, dv, dtype=torch.float32)
+    res = torch.empty(T, Hq, dv, dtype=torch.float32)
     rep = Hq // G
     for t in range(T):
         pos = int(tok_pos[t])
@@ -282,40 +318,44 @@ def sink_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, 
         if sink is not None:
             s = torch.cat([s, sink.float()[:, None]], dim=1)
         p = torch.softmax(s, dim=-1)[:, : js.numel()]
-        out[t] = torch.einsum("hn,nhd->hd", p, v)
-    out = out.reshape(T, Hq * dv)
+        res[t] = torch.einsum("hn,nhd->hd", p, v)
+    res = res.reshape(T, Hq * dv)
     if gate is not None:
-        out = out * torch.sigmoid(gate.float()).repeat_interleave(Hq * dv // gate.shape[1], dim=1)
-    return out.to(out_dtype)
+        res = res * torch.sigmoid(gate.float()).repeat_interleave(Hq * dv // gate.shape[1], dim=1)
+    return _out_rows(out, T, Hq * dv, out_dtype, q.device).copy_(res * out_scale)
 
 
 # ------------------------------------------------------------------------------------------------ short convolution
-def conv_silu(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], state: torch.Tensor,
-              seq_info: torch.Tensor, tok_seq: torch.Tensor) -> torch.Tensor:
-    """Short causal per-channel filter + SiLU over the rows ``x`` ``[T, C]`` of a ragged batch; ``w`` ``[C, taps]`` (last
-    column multiplies the current token), inputs before this batch's rows come from ``state`` ``[slots, taps-1, C]``,
-    inputs before a sequence's start are zero.  Returns fp32 ``[T, C]``; call :func:`conv_state_update` afterwards."""
+def conv_silu(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], state: Optional[torch.Tensor],
+              seq_info: torch.Tensor, tok_seq: torch.Tensor, in_bias: Optional[torch.Tensor] = None,
+              act: bool = True) -> torch.Tensor:
+    """Short causal per-channel filter + SiLU (not with ``act`` False) over the rows ``x`` ``[T, C]`` of a ragged batch; ``w``
+    ``[C, taps]`` (last column multiplies the current token), inputs before this batch's rows come from ``state`` ``[slots,
+    taps-1, C]`` (None for one tap), inputs before a sequence's start are zero; ``in_bias`` ``[C]`` is added to every input the
+    sequence has, ``bias`` to the sum.  Returns fp32 ``[T, C]``; call :func:`conv_state_update` afterwards."""
     T, C = x.shape
     taps = w.shape[1]
     if x.is_cuda:
         out = torch.empty(T, C, dtype=torch.float32, device=x.device)
-        _lib.call("sxb_conv_silu", _rows(x).data_ptr(), x.stride(0), w.data_ptr(), _lib.ptr(bias), state.data_ptr(),
-                  seq_info.data_ptr(), tok_seq.data_ptr(), out.data_ptr(), T, C, taps, _dt(x), _lib.stream_ptr())
+        _lib.call("sxb_conv_silu", _rows(x).data_ptr(), x.stride(0), w.data_ptr(), _lib.ptr(bias), _lib.ptr(state),
+                  seq_info.data_ptr(), tok_seq.data_ptr(), out.data_ptr(), T, C, taps, _lib.ptr(in_bias), int(act), _dt(x),
+                  _lib.stream_ptr())
         return out
     out = torch.empty(T, C, dtype=torch.float32)
     wf = w.float()
+    ib = 0.0 if in_bias is None else in_bias.float()
     for first, n, seen, slot in seq_info.tolist():
-        hist = state[slot].float() if seen > 0 else torch.zeros(taps - 1, C)
-        if 0 < seen < taps - 1:
-            hist = hist.clone()
-            hist[: taps - 1 - seen] = 0
-        full = torch.cat([hist, x[first: first + n].float()], dim=0)
+        hist = torch.zeros(taps - 1, C)
+        have = min(seen, taps - 1)
+        if have:
+            hist[taps - 1 - have:] = state[slot].float()[taps - 1 - have:] + ib
+        full = torch.cat([hist, x[first: first + n].float() + ib], dim=0)
         acc = torch.zeros(n, C)
         for j in range(taps):
             acc += wf[:, taps - 1 - j] * full[taps - 1 - j: taps - 1 - j + n]
         if bias is not None:
             acc += bias.float()
-        out[first: first + n] = torch.nn.functional.silu(acc)
+        out[first: first + n] = torch.nn.functional.silu(acc) if act else acc
     return out
 
 
@@ -392,26 +432,27 @@ def channel_decay_gates(a_raw: torch.Tensor, b_raw: torch.Tensor, A_log: torch.T
 
 
 def linear_recurrence(kvec: torch.Tensor, qvec: torch.Tensor, val: torch.Tensor, decay: torch.Tensor,
-                      beta: torch.Tensor, skip: Optional[torch.Tensor], state: torch.Tensor, seq_info: torch.Tensor,
+                      beta: Optional[torch.Tensor], skip: Optional[torch.Tensor], state: torch.Tensor, seq_info: torch.Tensor,
                       H: int, G: int, n: int, dv: int, delta: bool) -> torch.Tensor:
     """Per sequence and head, rows in order: ``S <- decay S``; ``u = beta (v - S^T k)`` (``delta``) or ``beta v``;
     ``S <- S + k u^T``; ``o = S^T q (+ skip[h] v)``.  ``kvec`` / ``qvec`` fp32 ``[T, G*n]`` and ``val`` fp32
     ``[T, H*dv]`` may be column slices (``kvec`` and ``qvec`` with one row pitch); ``state`` fp32 ``[slots, H, dv, n]`` is
     read (zero for a sequence that has seen no token) and written back.  ``decay`` fp32 ``[T, H]`` is one factor per
-    head; ``[T, H*n]`` one per head and key channel (it multiplies the state's entries of that channel).  Returns fp32
-    ``[T, H*dv]``."""
+    head; ``[T, H*n]`` one per head and key channel (it multiplies the state's entries of that channel); ``[H]`` one per head
+    for every row.  ``beta`` None: ones.  Returns fp32 ``[T, H*dv]``."""
     T = val.shape[0]
-    per_channel = decay.shape[1] == H * n and n > 1
+    fixed = decay.dim() == 1
+    per_channel = not fixed and decay.shape[1] == H * n and n > 1
     if val.is_cuda:
         if kvec.stride(0) != qvec.stride(0):
             raise ValueError("kvec and qvec must share their row pitch")
-        if not decay.is_contiguous() or decay.shape[1] not in (H, H * n):
-            raise ValueError("decay is a contiguous [T, H] or [T, H*n] tensor")
+        if not decay.is_contiguous() or decay.shape[-1] not in (H, H * n) or (fixed and decay.numel() != H):
+            raise ValueError("decay is a contiguous [T, H], [T, H*n] or [H] tensor")
         out = torch.empty(T, H * dv, dtype=torch.float32, device=val.device)
         _lib.call("sxb_linear_recurrence", _rows(kvec).data_ptr(), _rows(qvec).data_ptr(), kvec.stride(0),
-                  _rows(val).data_ptr(), val.stride(0), decay.data_ptr(), beta.data_ptr(), _lib.ptr(skip),
+                  _rows(val).data_ptr(), val.stride(0), decay.data_ptr(), _lib.ptr(beta), _lib.ptr(skip),
                   state.data_ptr(), out.data_ptr(), seq_info.data_ptr(), seq_info.shape[0], H, G, n, dv, int(delta),
-                  int(per_channel), _lib.stream_ptr())
+                  int(per_channel), int(fixed), _lib.stream_ptr())
         return out
     out = torch.empty(T, H, dv, dtype=torch.float32)
     rep = H // G
@@ -421,8 +462,11 @@ def linear_recurrence(kvec: torch.Tensor, qvec: torch.Tensor, val: torch.Tensor,
             k = kvec[t].reshape(G, n).repeat_interleave(rep, dim=0)                      # [H, n]
             q = qvec[t].reshape(G, n).repeat_interleave(rep, dim=0)
             v = val[t].reshape(H, dv)
-            S = S * (decay[t].reshape(H, 1, n) if per_channel else decay[t][:, None, None])
-            u = beta[t][:, None] * ((v - torch.einsum("hvn,hn->hv", S, k)) if delta else v)
+            a = decay if fixed else decay[t]
+            S = S * (a.reshape(H, 1, n) if per_channel else a[:, None, None])
+            u = (v - torch.einsum("hvn,hn->hv", S, k)) if delta else v
+            if beta is not None:
+                u = beta[t][:, None] * u
             S = S + u[:, :, None] * k[:, None, :]
             o = torch.einsum("hvn,hn->hv", S, q)
             if skip is not None:
@@ -433,22 +477,24 @@ def linear_recurrence(kvec: torch.Tensor, qvec: torch.Tensor, val: torch.Tensor,
 
 
 def group_norm_gate(y: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, group_size: int, eps: float,
-                    gate_first: bool, out_dtype: torch.dtype, sigmoid: bool = False) -> torch.Tensor:
+                    gate_first: bool, out_dtype: torch.dtype, sigmoid: bool = False, out: Optional[torch.Tensor] = None,
+                    out_scale: float = 1.0) -> torch.Tensor:
     """RMS norm over groups of ``group_size`` channels of fp32 ``y`` ``[T, C]`` with a SiLU gate ``[T, C]`` (column slice
     allowed) and a weight that repeats along the row.  ``gate_first``: ``norm(y * silu(gate)) * w``; else
-    ``norm(y) * w * silu(gate)``.  ``sigmoid``: the gate is ``sigmoid(gate)`` instead of ``silu(gate)``."""
+    ``norm(y) * w * silu(gate)``.  ``sigmoid``: the gate is ``sigmoid(gate)`` instead of ``silu(gate)``.  ``out`` (a column
+    slice is fine) receives the result, multiplied by ``out_scale`` before it is rounded."""
     T, C = y.shape
     if y.is_cuda:
-        out = torch.empty(T, C, dtype=out_dtype, device=y.device)
+        out = _out_rows(out, T, C, out_dtype, y.device)
         _lib.call("sxb_group_norm_gate", y.data_ptr(), _rows(gate).data_ptr(), gate.stride(0), w.data_ptr(), w.numel(),
-                  out.data_ptr(), T, C, group_size, float(eps), int(gate_first) | (2 if sigmoid else 0),
-                  _lib.dtype_code(out_dtype), _lib.stream_ptr())
+                  out.data_ptr(), T, C, group_size, float(eps), int(gate_first) | (2 if sigmoid else 0), out.stride(0),
+                  float(out_scale), _lib.dtype_code(out_dtype), _lib.stream_ptr())
         return out
     sg = torch.sigmoid(gate.float()) if sigmoid else torch.nn.functional.silu(gate.float())
     wf = w.float().repeat(C // w.numel())
     z = y * sg if gate_first else y
     z = _rms(z.reshape(T, C // group_size, group_size), eps).reshape(T, C) * wf
-    return (z if gate_first else z * sg).to(out_dtype)
+    return _out_rows(out, T, C, out_dtype, y.device).copy_((z if gate_first else z * sg) * out_scale)
 
 
 def gated_act_rows(x: torch.Tensor, act: str = "gelu", limit: float = 0.0) -> torch.Tensor:

@@ -12,12 +12,12 @@ from typing import Optional, Tuple
 import torch
 
 from ....native import lib as _lib
-from .mixer_ops import _rms, _rows
+from .mixer_ops import _rms, _rows, rotate_heads
 
 _lib.register({
     "sxb_resid_sum_step": "pppppp" "ff" "pppppppppp" "iii" "i" "p",
     "sxb_norm_filter_rows": "pppppppppp" "iiii" "i" "p",
-    "sxb_rope_append": "p" "l" "iii" "pppppppppp" "iiiiiiiii" "f" "i" "p",
+    "sxb_rope_append": "p" "l" "iii" "pppppppppp" "iiiiiiiii" "ff" "i" "p",
     "sxb_removal_prepare": "p" "l" "iiiii" "pppp" "iiii" "ff" "i" "p",
     "sxb_removal_recurrence": "pppp" "iiii" "p",
 })
@@ -126,28 +126,14 @@ def open_parallel_layer(resid: torch.Tensor, add: Optional[StreamSum], w_mix: to
 
 
 # ------------------------------------------------------------------------------------------------ attention rows
-def _turn(x: torch.Tensor, pos: torch.Tensor, inv_freq: torch.Tensor, interleaved: bool) -> torch.Tensor:
-    half = inv_freq.numel()
-    ang = pos.float()[:, None, None] * inv_freq.float()
-    c, s = ang.cos(), ang.sin()
-    out = x.clone()
-    if interleaved:
-        u, v = x[..., 0: 2 * half: 2], x[..., 1: 2 * half: 2]
-        out[..., 0: 2 * half: 2], out[..., 1: 2 * half: 2] = u * c - v * s, v * c + u * s
-    else:
-        u, v = x[..., :half], x[..., half: 2 * half]
-        out[..., :half], out[..., half: 2 * half] = u * c - v * s, v * c + u * s
-    return out
-
-
 def rope_append(proj: torch.Tensor, q0: int, k0: int, v0: int, q_w: Optional[torch.Tensor], k_w: Optional[torch.Tensor],
                 inv_freq: torch.Tensor, interleaved: bool, q_scale: Optional[torch.Tensor], kcache: torch.Tensor,
                 vcache: torch.Tensor, tok_seq: torch.Tensor, tok_pos: torch.Tensor, tables: torch.Tensor, Hq: int, G: int,
-                d: int, dv: int, eps: float) -> torch.Tensor:
+                d: int, dv: int, eps: float, amp: float = 1.0) -> torch.Tensor:
     """q (``Hq d`` columns at ``q0``), k (``G d`` at ``k0``) and v (``G dv`` at ``v0``; ``v0 = k0``: the values are the projected
     keys, untouched) of projection rows.  With ``q_w`` / ``k_w`` (``[Hq d]`` / ``[G d]``) the whole row of q / k is divided by its
     root mean square and multiplied by the weight.  The first ``2 len(inv_freq)`` channels of every head turn by ``pos *
-    inv_freq[i]``: pairs ``(2i, 2i+1)`` if ``interleaved``, else ``(i, i + len(inv_freq))``.  Returns q fp32 ``[T, Hq, d]`` times
+    inv_freq[i]``: pairs ``(2i, 2i+1)`` if ``interleaved``, else ``(i, i + len(inv_freq))``, cos and sin times ``amp``.  Returns q fp32 ``[T, Hq, d]`` times
     ``q_scale`` (fp32 ``[Hq]``); k and v go to the paged caches ``[pages, block, G, d | dv]``."""
     T = proj.shape[0]
     bs = kcache.shape[1]
@@ -159,7 +145,7 @@ def rope_append(proj: torch.Tensor, q0: int, k0: int, v0: int, q_w: Optional[tor
         _lib.call("sxb_rope_append", _rows(proj).data_ptr(), proj.stride(0), int(q0), int(k0), int(v0), _lib.ptr(q_w),
                   _lib.ptr(k_w), inv_freq.data_ptr() if n_rot else None, _lib.ptr(q_scale), q.data_ptr(), kcache.data_ptr(),
                   vcache.data_ptr(), tok_seq.data_ptr(), tok_pos.data_ptr(), tables.data_ptr(), T, tables.shape[1], bs, Hq, G,
-                  d, dv, n_rot, int(interleaved), float(eps), _lib.dtype_code(proj.dtype), _lib.stream_ptr())
+                  d, dv, n_rot, int(interleaved), float(eps), float(amp), _lib.dtype_code(proj.dtype), _lib.stream_ptr())
         return q
     x = proj.float()
     q, k = x[:, q0: q0 + Hq * d], x[:, k0: k0 + G * d]
@@ -168,8 +154,8 @@ def rope_append(proj: torch.Tensor, q0: int, k0: int, v0: int, q_w: Optional[tor
         q = _rms(q, eps) * q_w.float()
     if k_w is not None:
         k = _rms(k, eps) * k_w.float()
-    q = _turn(q.reshape(T, Hq, d), tok_pos, inv_freq, interleaved)
-    k = _turn(k.reshape(T, G, d), tok_pos, inv_freq, interleaved)
+    q = rotate_heads(q.reshape(T, Hq, d), tok_pos, inv_freq, interleaved, amp)
+    k = rotate_heads(k.reshape(T, G, d), tok_pos, inv_freq, interleaved, amp)
     if q_scale is not None:
         q = q * q_scale.float()[:, None]
     page = tables[tok_seq.long(), (tok_pos // bs).long()].long()

@@ -1,14 +1,15 @@
 """Ragged-batch model for hybrid layer stacks: every layer names its own token mixer — attention over the paged cache
 (per-head keys and values, or one latent vector per token), a gated-delta-rule (one decay per head, or per head and
-key channel, or separate decay and removal vectors), state-space-duality or matrix-memory LSTM recurrence, or two of these side
-by side — and may or may not have a feed-forward (gated, biased, or a mixture of experts); a span of layers can be executed several times in a row with the same weights, and
+key channel, or separate decay and removal vectors), state-space-duality, matrix-memory LSTM, lightning or gated linear
+attention recurrence, a linear recurrent unit, or two of these side by side — and may or may not have a feed-forward (gated, biased, or a mixture of experts); a span of layers can be executed several times in a row with the same weights, and
 single layers can borrow another layer's weights, every execution with its own cache or state.
 
 The stack is data (:class:`HybridSpec`), as :class:`~.inference_transformer_base.ArchSpec` is for the uniform
 transformer family; per-architecture policies (``fomalix/policy.py``) fill it from a checkpoint's configuration and fuse
 the checkpoint's tensors into the projection layouts the mixer modules declare.
 
-Four layer forms (``HybridSpec.block_form``).  ``"sandwich"``: ``x += post_norm(sublayer(pre_norm(x)))``.
+Four layer forms (``HybridSpec.block_form``).  ``"sandwich"``: ``x += post_norm(sublayer(pre_norm(x)))`` (with
+``norm_weight_offset`` all norms multiply by ``offset + w``).
 ``"pre_scaled"``: ``x += m * sublayer(pre_norm(x))`` with one multiplier ``m`` for the whole stack (with ``layer_scale``
 also a learned scale per layer, sublayer and channel: ``x += m * ls (.) sublayer(pre_norm(x))``; with
 ``norm_weight_offset`` the norms multiply by ``offset + w``), and optionally a
@@ -50,7 +51,8 @@ from .inference_transformer_base import DSInferenceModelBase, LayerWeights
 
 @dataclass
 class HybridLayerSpec:
-    # "attention" | "rotary_attention" | "latent_attention" | "delta" | "channel_delta" | "removal_delta" | "ssd" | "mlstm" | "pair"
+    # "attention" | "rotary_attention" | "latent_attention" | "delta" | "channel_delta" | "removal_delta" | "ssd" | "mlstm" |
+    # "lightning" | "channel_decay" | "lru" (n_heads blocks of key_dim channels) | "pair"
     kind: str
     n_heads: int
     n_heads_kv: int                             # key/value heads (attention), key/query heads (delta), groups (ssd)
@@ -99,6 +101,8 @@ class HybridLayerSpec:
     moe_correction: bool = False
     moe_groups: int = 1
     moe_keep_groups: int = 1
+    moe_group_rank: str = "max"
+    moe_plain_scores: bool = False              # the group-limited choice's weights are not divided by their sum
     moe_scale: float = 1.0
     moe_identity: int = 0
     ff_limit: float = 0.0
@@ -110,9 +114,13 @@ class HybridLayerSpec:
     values_from_keys: bool = False
     unit_sink: bool = False
     head_scale: bool = False
-    decay_rate: float = 1.0                     # removal delta: decay = exp(-decay_rate * sigmoid(.))
-    # pair: two mixers that read the same input; the layer's mixer output is half the sum of their RMS-normed outputs
+    decay_rate: float = 1.0                     # removal delta: decay = exp(-decay_rate * sigmoid(.)); lru: exponent's factor
+    head_decay: Optional[Tuple[float, ...]] = None      # lightning: the decay of every head
+    decay_tau: float = 1.0                      # channel_decay: decay = sigmoid(.)^(1 / tau)
+    # pair: two mixers that read the same input; the layer's mixer output is half the sum of their RMS-normed outputs, or with
+    # ``pair_scales`` the sum of their outputs times one factor each
     parts: Optional[Tuple["HybridLayerSpec", "HybridLayerSpec"]] = None
+    pair_scales: Optional[Tuple[float, float]] = None
 
 
 @dataclass
@@ -132,7 +140,7 @@ class HybridSpec:
     residual_mult: float = 1.0                  # pre_scaled: what every sublayer's output is multiplied by
     token_side_dim: int = 0                     # pre_scaled: channels per layer of the per-layer token input (0: none)
     layer_scale: bool = False                   # pre_scaled: every sublayer's output times a per-channel ``ls1`` / ``ls2``
-    norm_weight_offset: float = 0.0             # pre_scaled: norm weights are ``offset + w`` (1: stored around zero)
+    norm_weight_offset: float = 0.0             # pre_scaled, sandwich: norm weights are ``offset + w`` (1: stored around zero)
     logit_scale: float = 1.0
     logit_softcap: float = 0.0                  # > 0: logits <- cap * tanh(logits / cap)
     input_conv_taps: int = 0                    # taps of the filter in front of every sublayer (post_scaled) or mixer (parallel)
@@ -170,7 +178,9 @@ class DSHybridModel(DSInferenceModelBase):
     ``moe_correction`` (fp32), ``moe_w1``, ``moe_w2``.  Two entries of ``layers`` may be one object (borrowed weights).
     Parallel stacks: ``norm1``, ``norm2``, ``filter1`` (``[taps, width]``); rotary attention ``q_norm`` / ``k_norm``,
     ``q_head_scale`` (fp32); a pair has one ``w_in`` for both mixers and ``parts``, two :class:`LayerWeights` with the mixers'
-    tensors, ``wo`` and ``out_norm``; removal delta ``w0``, ``a_bias`` (fp32), ``w2`` (``[rank, heads * dim]``), ``norm``."""
+    tensors, ``wo`` and ``out_norm``; removal delta ``w0``, ``a_bias`` (fp32), ``w2`` (``[rank, heads * dim]``), ``norm``.  A pair
+    with ``pair_scales`` has ONE ``wo`` over both results side by side: the first mixer's projection columns end at ``cut``,
+    the second's input columns of ``wo`` start at ``wo_cut``, ``parts[j].wo_width`` columns belong to mixer ``j``."""
 
     def __init__(self, spec: HybridSpec, weights: Dict, engine_config: RaggedInferenceEngineConfig, state_manager=None,
                  base_mp_group=None) -> None:
@@ -232,7 +242,7 @@ class DSHybridModel(DSInferenceModelBase):
                     score_function=L.moe_score, weight_input=L.moe_weight_input, router_dtype=DtypeEnum.fp32,
                     router_bias=L.router_bias, shared_features=L.shared_ff_dim,
                     score_correction=L.moe_correction, n_groups=L.moe_groups, keep_groups=L.moe_keep_groups,
-                    score_scale=L.moe_scale, identity_experts=L.moe_identity, activation_limit=L.ff_limit), ec)
+                    group_rank=L.moe_group_rank, plain_group_scores=L.moe_plain_scores, score_scale=L.moe_scale, identity_experts=L.moe_identity, activation_limit=L.ff_limit), ec)
             self.moes.append(moe)
             self.mixers.append(tuple(self._build_mixer(part) for part in L.parts) if L.kind == "pair" else self._build_mixer(L))
         self._state_cfg = StatePoolConfig()
@@ -274,6 +284,10 @@ class DSHybridModel(DSInferenceModelBase):
                 rotary_scaling=None if L.rot_scaling is None else RotaryScalingConfig(
                     factor=L.rot_scaling[0], original=L.rot_scaling[1], fast=L.rot_scaling[2],
                     slow=L.rot_scaling[3])), ec)
+        scaling = None if L.rot_scaling is None else RotaryScalingConfig(
+            factor=L.rot_scaling[0], original=L.rot_scaling[1], fast=L.rot_scaling[2], slow=L.rot_scaling[3])
+        rotation = (PositionalEmbeddingType.none if L.rot_dims == 0 else
+                    PositionalEmbeddingType.rotate_every_other if L.rot_interleaved else PositionalEmbeddingType.rotate_half)
         if L.kind == "attention" and (L.conv_taps > 1 or L.qk_norm_weight or L.dist_rows > 0 or L.out_gate
                                         or L.q_temp_coef != 0.0):
             mask = (MaskingType.chunked if L.chunk_size > 0 else
@@ -283,8 +297,10 @@ class DSHybridModel(DSInferenceModelBase):
                 v_head_size=L.value_dim, max_sequences=sm.max_ragged_sequence_count, scale_factor=L.attn_scale,
                 input_dtype=dt, output_dtype=dt, masking_type=mask,
                 masking_args={"size": L.chunk_size or L.window} if mask != MaskingType.causal else {},
-                positional_embedding_type=(PositionalEmbeddingType.distance_bias if L.dist_rows > 0
-                                           else PositionalEmbeddingType.none),
+                positional_embedding_type=PositionalEmbeddingType.distance_bias if L.dist_rows > 0 else rotation,
+                positional_embedding_config=RotateHalfConfig(theta_base=L.rot_base, rotate_dim=L.rot_dims,
+                                                             freq_divisor=L.rot_divisor),
+                rotary_scaling=scaling,
                 distance_bias=DistanceBiasConfig(rows=L.dist_rows, far=L.dist_far) if L.dist_rows > 0 else None,
                 qk_norm_eps=s.norm_eps, qkv_conv_taps=L.conv_taps, qk_norm_weight=L.qk_norm_weight,
                 q_temp_coef=L.q_temp_coef, q_temp_every=L.q_temp_every, output_gate=L.out_gate), ec)
@@ -303,19 +319,17 @@ class DSHybridModel(DSInferenceModelBase):
                 max_sequences=sm.max_ragged_sequence_count, scale_factor=L.attn_scale, input_dtype=dt, output_dtype=dt,
                 masking_type=MaskingType.sliding_window if L.window > 0 else MaskingType.causal,
                 masking_args={"size": L.window} if L.window > 0 else {},
-                positional_embedding_type=(PositionalEmbeddingType.none if L.rot_dims == 0 else
-                                           PositionalEmbeddingType.rotate_every_other if L.rot_interleaved else
-                                           PositionalEmbeddingType.rotate_half),
+                positional_embedding_type=rotation,
                 positional_embedding_config=RotateHalfConfig(theta_base=L.rot_base, rotate_dim=L.rot_dims,
                                                              freq_divisor=L.rot_divisor),
-                qk_norm_eps=s.norm_eps, split_cache=True, qk_row_norm=L.qk_row_norm, values_from_keys=L.values_from_keys,
+                rotary_scaling=scaling, qk_norm_eps=s.norm_eps, split_cache=True, qk_row_norm=L.qk_row_norm, values_from_keys=L.values_from_keys,
                 unit_sink=L.unit_sink, sink=L.sink, q_head_scale=L.head_scale, output_gate=L.out_gate,
                 output_gate_per_head=L.gate_per_head), ec)
         return heuristics.instantiate_recurrent_mixer(DSRecurrentMixerConfig(
             max_tokens=mt, kind=L.kind, model_dim=s.model_dim, n_heads=L.n_heads, n_heads_kv=L.n_heads_kv,
             key_dim=L.key_dim, value_dim=L.value_dim, conv_taps=L.conv_taps, norm_groups=L.norm_groups,
-            gate_cap=L.gate_cap, decay_rate=L.decay_rate, eps=s.norm_eps, max_sequences=sm.max_ragged_sequence_count,
-            input_dtype=dt, output_dtype=dt), ec)
+            gate_cap=L.gate_cap, decay_rate=L.decay_rate, head_decay=L.head_decay, decay_tau=L.decay_tau, eps=s.norm_eps,
+            max_sequences=sm.max_ragged_sequence_count, input_dtype=dt, output_dtype=dt), ec)
 
     def _plan_memory(self, key, L: HybridLayerSpec, mod, shapes: List) -> None:
         """Cache and state entries of one execution of a mixer (``key``: the run, or (run, part) in a pair)."""
@@ -387,26 +401,29 @@ class DSHybridModel(DSInferenceModelBase):
                 h = M.bias_act_rows(self.linear(x, lw.w_up), lw.b_up, L.ff_activation)
             return F.linear(h, lw.w_down, lw.b_down)
         h = self.linear(x, lw.w_gate_up)
-        if h.is_cuda and h.dtype == torch.bfloat16 and L.ff_dim % 8 == 0:
+        if L.ff_activation != "clamped_swish" and h.is_cuda and h.dtype == torch.bfloat16 and L.ff_dim % 8 == 0:
             h = F.gated_act(h, L.ff_activation)
         else:
-            h = M.gated_act_rows(h, L.ff_activation)
+            h = M.gated_act_rows(h, L.ff_activation, L.ff_limit)
         return self.linear(h, lw.w_down)
 
-    def _mix(self, key, L: HybridLayerSpec, mod, lw: LayerWeights, proj: torch.Tensor, batch) -> torch.Tensor:
-        """A mixer on its projection columns, before its output projection."""
+    def _mix(self, key, L: HybridLayerSpec, mod, lw: LayerWeights, proj: torch.Tensor, batch, **out) -> torch.Tensor:
+        """A mixer on its projection columns, before its output projection (``out``: where its result goes and the factor on
+        it, for the mixers that take them)."""
         sm = self.state_manager
         if L.kind == "attention" and hasattr(mod, "filtered_channels"):
             states = self._state_of_run.get(key, ())
             return mod(proj, sm.get_cache(self._cache_of_run[key]), batch, None, lw,
-                       sm.get_state(states[0]) if states else None)
+                       sm.get_state(states[0]) if states else None, **out)
         if L.kind == "attention":
             return mod(proj, sm.get_cache(self._cache_of_run[key]), batch, None, lw.b_in, lw.sink)
         if L.kind in ("latent_attention", "rotary_attention"):
-            return mod(proj, sm.get_cache(self._cache_of_run[key]), batch, None, lw)
-        return mod(proj, lw, tuple(sm.get_state(e) for e in self._state_of_run[key]), batch)
+            return mod(proj, sm.get_cache(self._cache_of_run[key]), batch, None, lw, **out)
+        return mod(proj, lw, tuple(sm.get_state(e) for e in self._state_of_run[key]), batch, **out)
 
     def _mixer(self, r: int, li: int, lw: LayerWeights, x: torch.Tensor, batch) -> torch.Tensor:
+        if self.spec.layers[li].kind == "pair":
+            return self._mixer_sum(r, li, lw, x, batch)
         ctx = self._mix(r, self.spec.layers[li], self.mixers[li], lw, self.linear(x, lw.w_in), batch)
         return self.linear(ctx, lw.wo)
 
@@ -418,6 +435,21 @@ class DSHybridModel(DSInferenceModelBase):
         a, b = (self.linear(self._mix((r, j), L.parts[j], mods[j], lw.parts[j], cols, batch), lw.parts[j].wo)
                 for j, cols in enumerate((proj[:, :cut], proj[:, cut:])))
         return P.StreamSum(a=a, wa=lw.parts[0].out_norm, b=b, wb=lw.parts[1].out_norm, mult=0.5)
+
+    def _mixer_sum(self, r: int, li: int, lw: LayerWeights, x: torch.Tensor, batch) -> torch.Tensor:
+        """``s0 * mixer0(x) + s1 * mixer1(x)``: one fused projection in, and one out of both mixers' results side by side (the
+        factors enter where a mixer rounds its result), so that the sum is formed in the product's accumulator."""
+        L, mods = self.spec.layers[li], self.mixers[li]
+        proj = self.linear(x, lw.w_in)
+        cut = lw.cut
+        widths = [part.wo_width for part in lw.parts]
+        both = (torch.empty if lw.wo.shape[1] == sum(widths) else torch.zeros)(x.shape[0], lw.wo.shape[1], dtype=x.dtype,
+                                                                              device=x.device)
+        for j, cols in enumerate((proj[:, :cut], proj[:, cut:])):
+            at = j * lw.wo_cut
+            self._mix((r, j), L.parts[j], mods[j], lw.parts[j], cols, batch, out=both[:, at: at + widths[j]],
+                      out_scale=L.pair_scales[j])
+        return self.linear(both, lw.wo)
 
     def _filtered(self, x: torch.Tensor, w: torch.Tensor, entry: int, batch) -> torch.Tensor:
         """What a sublayer of a post-scaled layer reads: ``x + filter(x)`` in the activation dtype; the sequence's
@@ -507,7 +539,12 @@ class DSHybridModel(DSInferenceModelBase):
         resid = resid.index_select(0, rows)
         _, x = self.norm(resid, None if y is None else y.index_select(0, rows), W["final_norm_w"], None, post, None, m,
                          False, ls, off)
-        logits = self.linear(x, W["unembed"])[:, : s.vocab_size].float().contiguous()
+        return self._logits(x)
+
+    def _logits(self, x: torch.Tensor) -> torch.Tensor:
+        """fp32 logits of normed rows: head, factor, soft cap."""
+        s = self.spec
+        logits = self.linear(x, self.weights["unembed"])[:, : s.vocab_size].float().contiguous()
         if s.logit_scale != 1.0 or s.logit_softcap > 0.0:
             M.scale_softcap_(logits, s.logit_scale, s.logit_softcap)
         return logits
@@ -553,17 +590,22 @@ class DSHybridModel(DSInferenceModelBase):
             return self._forward_pre_scaled(batch)
         resid = self.embed(batch, W["embed"])
         first = resid.clone() if any(again for _, again in self._runs) else None
+        off = dict(gamma_offset=s.norm_weight_offset, post_offset=s.norm_weight_offset)
         y = post = None                     # output of the last sublayer and its post-norm weight, not yet added
         for r, (li, again) in enumerate(self._runs):
             lw, L = W["layers"][li], s.layers[li]
-            _, x = self.norm(resid, y, lw.norm1, None, post, first if again else None)
+            _, x = self.norm(resid, y, lw.norm1, None, post, first if again else None, **off)
             y, post = self._mixer(r, li, lw, x, batch), lw.norm1b
             if L.ff_dim > 0:
-                _, x = self.norm(resid, y, lw.norm2, None, post, None)
+                _, x = self.norm(resid, y, lw.norm2, None, post, None, **off)
                 y, post = self._feed_forward(L, lw, x, li), lw.norm2b
+            if self.layer_outputs is not None:
+                self.norm(resid, y, None, None, post, None, **off)
+                y = post = None
+                self.layer_outputs.append(resid.clone())
         rows = batch.last_token_index().long()
         if rows.numel() == 0:               # a step that only advances caches and states
             return torch.empty(0, s.vocab_size, dtype=torch.float32, device=resid.device)
         resid = resid.index_select(0, rows)
-        _, x = self.norm(resid, None if y is None else y.index_select(0, rows), W["final_norm_w"], None, post, None)
-        return self.linear(x, W["unembed"])[:, : s.vocab_size].float()
+        _, x = self.norm(resid, None if y is None else y.index_select(0, rows), W["final_norm_w"], None, post, None, **off)
+        return self._logits(x)

@@ -277,9 +277,10 @@ from .kekopel import KekopelPolicy  # noqa: E402
 from .ridazen import RidazenPolicy  # noqa: E402
 from .pifazen import PifazenPolicy  # noqa: E402
 from .vezodra import VezodraPolicy  # noqa: E402
+from .sudupel import SudupelPolicy  # noqa: E402
 
 POLICIES = {"fomalix": FomalixPolicy, "kekopel": KekopelPolicy, "ridazen": RidazenPolicy, "pifazen": PifazenPolicy,
-            "vezodra": VezodraPolicy,
+            "vezodra": VezodraPolicy, "sudupel": SudupelPolicy,
             "llama": Llama2Policy, "mistral": MistralPolicy, "mixtral": MixtralPolicy, "falcon": FalconPolicy,
             "opt": OPTPolicy, "phi": PhiPolicy, "phi3": Phi3Policy, "qwen": QwenPolicy, "qwen2": Qwen2Policy,
             "qwen2_moe": Qwen2MoePolicy}

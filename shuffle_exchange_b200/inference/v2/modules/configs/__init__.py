@@ -1,6 +1,6 @@
 """Module configs (reference ``inference/v2/modules/configs/*``)."""
 from enum import Enum
-from typing import Dict, Optional
+from typing import Dict, Optional, Tuple
 
 from ...inference_utils import ActivationType, DtypeEnum, NormTypeEnum
 from ..ds_module import DSModuleConfig
@@ -131,12 +131,15 @@ class DSMoEConfig(DSModuleConfig):
     # one more router row (the row after the experts' rows) and added.
     shared_features: int = 0
     # Group-limited choice: the router has ``n_experts + identity_experts`` outputs in ``n_groups`` equal groups of
-    # neighbours; the winners are the ``top_k`` largest ``score + correction`` inside the ``keep_groups`` groups whose
-    # best member is largest; the weights are the winners' plain scores / their sum * ``score_scale``.  The last
-    # ``identity_experts`` outputs stand for experts that return their input (they have no weights).
+    # neighbours; the winners are the ``top_k`` largest ``score + correction`` inside the ``keep_groups`` groups that rank
+    # first, by their best member (``group_rank`` "max") or the sum of their two best ("top2"); the weights are the winners'
+    # plain scores / their sum (``plain_group_scores``: not divided) * ``score_scale``.  The last ``identity_experts`` outputs stand for
+    # experts that return their input (they have no weights).
     score_correction: bool = False
     n_groups: int = 1
     keep_groups: int = 1
+    group_rank: str = "max"
+    plain_group_scores: bool = False
     score_scale: float = 1.0
     identity_experts: int = 0
     activation_limit: float = 0.0         # ActivationType.CLAMPED_SWIGLU: the clamp
@@ -171,7 +174,12 @@ class DSRecurrentMixerConfig(DSModuleConfig):
     (exponential input gate, sigmoid forget gate in log space, both capped by ``gate_cap``, a running maximum that
     keeps the exponentials in range, a normaliser state, per-head unit-RMS and a sigmoid output gate; no convolution).
     ``"removal_delta"``: a delta rule whose decay, and whose rate of removing what a key has stored, are vectors over the key
-    channels of every head (no convolution, key and value sizes equal; ``decay_rate`` bounds the decay from below)."""
+    channels of every head (no convolution, key and value sizes equal; ``decay_rate`` bounds the decay from below).
+    ``"lightning"``: SiLU on q, k and v, one fixed decay per head (``head_decay``), no write strength, an RMS norm over all heads
+    at once and a sigmoid gate.  ``"channel_decay"``: gated linear attention, a decay per head and key channel from a two-step
+    projection (``sigmoid(.)^(1 / decay_tau)``), per-head RMS norm, SiLU gate.  ``"lru"``: a gated linear recurrent unit of
+    ``n_heads`` equal blocks of ``key_dim`` channels (an elementwise state instead of a matrix per head) behind a filter of
+    ``conv_taps`` taps; ``decay_rate`` is the exponent's factor."""
     kind: str
     model_dim: int
     n_heads: int
@@ -181,7 +189,9 @@ class DSRecurrentMixerConfig(DSModuleConfig):
     conv_taps: int = 1
     norm_groups: int = 1
     gate_cap: float = 0.0                 # mlstm: gate pre-activations pass cap * tanh(x / cap)
-    decay_rate: float = 1.0               # removal_delta: decay = exp(-decay_rate * sigmoid(.))
+    decay_rate: float = 1.0               # removal_delta: decay = exp(-decay_rate * sigmoid(.)); lru: see there
+    head_decay: Optional[Tuple[float, ...]] = None
+    decay_tau: float = 1.0
     eps: float = 1e-5
     unit_norm_eps: float = 1e-6
     max_sequences: int = 1

@@ -22,7 +22,7 @@ def instantiate_attention(attention_config: DSSelfAttentionConfig,
     if not DSSelfAttentionRegistry.registry[name].supports_config(attention_config):
         name = "sink_chunked_attention"       # chunk-local mask, sink logit, q/k unit norm or narrower value heads
     if not DSSelfAttentionRegistry.registry[name].supports_config(attention_config):
-        name = "filtered_bias_attention"      # filtered projections, weighted q/k norm, distance bias, output gate
+        name = "filtered_bias_attention"      # filtered projections, weighted q/k norm, rotation, distance bias, output gate
     if not DSSelfAttentionRegistry.registry[name].supports_config(attention_config):
         name = "rotary_sink_attention"        # rotated heads with split caches, whole-row norms, values taken from the keys
     return DSSelfAttentionRegistry.instantiate_config(ConfigBundle(name=name, config=attention_config))
@@ -69,10 +69,11 @@ def instantiate_unembed(unembed_config: DSUnembedConfig, engine_config: RaggedIn
 def instantiate_recurrent_mixer(mixer_config: DSRecurrentMixerConfig,
                                 engine_config: RaggedInferenceEngineConfig) -> DSRecurrentMixerBase:
     name = {"delta": "gated_delta_mixer", "ssd": "ssd_mixer", "mlstm": "mlstm_mixer",
-            "channel_delta": "channel_delta_mixer", "removal_delta": "removal_delta_mixer"}.get(mixer_config.kind)
+            "channel_delta": "channel_delta_mixer", "removal_delta": "removal_delta_mixer", "lightning": "lightning_mixer",
+            "channel_decay": "gated_linear_mixer", "lru": "linear_recurrent_unit"}.get(mixer_config.kind)
     if name is None:
         raise ValueError(f"Unknown recurrent mixer kind {mixer_config.kind!r}; expected 'delta', 'channel_delta', "
-                         "'removal_delta', 'ssd' or 'mlstm'")
+                         "'removal_delta', 'ssd', 'mlstm', 'lightning', 'channel_decay' or 'lru'")
     return DSRecurrentMixerRegistry.instantiate_config(ConfigBundle(name=name, config=mixer_config))
 
 

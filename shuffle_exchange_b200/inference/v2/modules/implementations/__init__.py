@@ -18,7 +18,7 @@
  ``fp32_scaled_post_rms``     fp32 stream += scale (.) rms_norm(sublayer output) * gain (+ mixture of all layers' streams)
  ``fp32_sandwich_rms``        fp32 residual += post-norm(sublayer output); next pre-norm, one kernel
  ``filtered_bias_attention``  q | k | v through a short causal filter with carried inputs, weighted per-head RMS norm,
-                              query temperature, learned distance-bucket bias on the scores, sigmoid output gate
+                              query temperature, rotation or a learned distance-bucket bias on the scores, sigmoid output gate
  ``gated_delta_mixer`` / ``ssd_mixer``   short convolutions with carried inputs + linear recurrence with a matrix
                               state per (sequence slot, head) + gated group norm
  ``channel_delta_mixer``      the delta rule with a separate decay for every key channel of every head and a sigmoid output gate, both
@@ -26,6 +26,9 @@
  ``rotary_sink_attention``    rotation in either pairing, whole-row q/k norm, values that may be the unrotated keys, causal or
                               windowed softmax that may add one to its denominator, a scale and an output gate per head
  ``removal_delta_mixer``      delta rule with a decay and a removal rate per head and key channel
+ ``lightning_mixer``          decayed sum of outer products, one fixed decay per head, norm over all heads, sigmoid gate
+ ``gated_linear_mixer``       decayed sum of outer products with a decay per head and key channel, per-head norm, SiLU gate
+ ``linear_recurrent_unit``    elementwise gated recurrence behind a short filter, block-diagonal gates, GELU branch
 =========================  =======================================================================================
 """
 from __future__ import annotations
@@ -42,6 +45,7 @@ from ...inference_utils import ActivationType, DtypeEnum, NormTypeEnum, is_gated
 from ...kernels import ragged_ops as R
 from ...kernels import mixer_ops as M
 from ...kernels import parallel_ops as P
+from ...kernels import gated_ops as Gt
 from ..configs import (DSEmbeddingsConfig, DSLinearConfig, DSMoEConfig, DSNormConfig, DSRecurrentMixerConfig,
                        DSSelfAttentionConfig, DSUnembedConfig, MaskingType, PositionalEmbeddingType)
 from ..interfaces import (DSEmbeddingBase, DSEmbeddingRegistry, DSLinearBase, DSLinearRegistry, DSMoEBase,
@@ -80,6 +84,38 @@ def _apply_activation(y: torch.Tensor, bias: Optional[torch.Tensor], act: Activa
     return F.bias_act(y, bias, _act_name(act))
 
 
+def scaled_rotary_table(n_rot: int, base: float, scaling=None, divisor: float = 1.0) -> Tuple[torch.Tensor, float]:
+    """fp32 angular frequencies ``base^(-2i / n_rot) / divisor`` of the ``n_rot / 2`` pairs and the factor on cos and sin.  With
+    ``scaling`` (:class:`RotaryScalingConfig`): let ``pair(t) = n_rot ln(original / (2 pi t)) / (2 ln base)`` be the (fractional)
+    pair that makes ``t`` turns over the original context, ``lo = max(floor(pair(fast)), 0)``, ``hi = min(ceil(pair(slow)),
+    n_rot - 1)`` and ``w_i = min(1, max(0, (i - lo) / max(hi - lo, 0.001)))``; pair ``i`` turns at ``f_i (1 - w_i) + w_i f_i /
+    factor`` and the amplitude is ``0.1 ln(factor) + 1``.  Evaluated in float64, stored as float32."""
+    i = torch.arange(0, n_rot, 2, dtype=torch.float64) / 2.0
+    f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / max(n_rot, 1)) / divisor
+    amp = 1.0
+    if scaling is not None and n_rot > 0:
+        def pair(turns: float) -> float:
+            return n_rot * math.log(scaling.original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+        lo = max(math.floor(pair(scaling.fast)), 0)
+        hi = min(math.ceil(pair(scaling.slow)), n_rot - 1)
+        ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        f = f / scaling.factor * ramp + f * (1.0 - ramp)
+        amp = 0.1 * math.log(scaling.factor) + 1.0
+    return f.to(torch.float32), float(amp)
+
+
+def rotated_channels(config: DSSelfAttentionConfig) -> Tuple[int, float, float, bool]:
+    """(channels of a head that turn, base, frequency divisor, interleaved pairs) of a rotated attention."""
+    pe, rot = PositionalEmbeddingType(config.positional_embedding_type), config.positional_embedding_config
+    n_rot = 0
+    if pe in (PositionalEmbeddingType.rotate_half, PositionalEmbeddingType.rotate_every_other):
+        n_rot = config.head_size if rot is None or rot.rotate_dim is None else rot.rotate_dim
+    if n_rot % 2 or n_rot > config.head_size:
+        raise ValueError(f"cannot rotate {n_rot} of {config.head_size} channels in pairs")
+    return (n_rot, 10000.0 if rot is None else rot.theta_base, 1.0 if rot is None else rot.freq_divisor,
+            pe == PositionalEmbeddingType.rotate_every_other)
+
+
 # ============================================================================================ attention
 @DSSelfAttentionRegistry.register_module
 class DSDenseBlockedAttention(DSSelfAttentionBase):
@@ -91,6 +127,8 @@ class DSDenseBlockedAttention(DSSelfAttentionBase):
     @staticmethod
     def supports_config(config: DSSelfAttentionConfig) -> bool:
         if MaskingType(config.masking_type) != MaskingType.causal or config.split_cache:
+            return False
+        if config.qkv_conv_taps > 1 or config.qk_norm_weight or config.rotary_scaling is not None or config.output_gate:
             return False
         if config.sink or config.qk_unit_rms or config.v_head_size not in (None, config.head_size):
             return False
@@ -297,8 +335,9 @@ class DSMultiGemmMoE(DSMoEBase):
             raise ValueError(f"the router has {logits.shape[1]} outputs for {c.n_experts} experts and {n_id} identity experts")
         if c.score_correction or c.n_groups > 1 or c.score_scale != 1.0 or n_id > 0:
             scores, assign, offsets, counts = moe_ops.top_k_gating(
-                logits, c.top_k, score_function=c.score_function, correction=correction if c.score_correction else None,
-                n_groups=c.n_groups, keep_groups=c.keep_groups, scale=c.score_scale)
+                logits, c.top_k, renormalize=not c.plain_group_scores, score_function=c.score_function,
+                correction=correction if c.score_correction else None, n_groups=c.n_groups, keep_groups=c.keep_groups,
+                scale=c.score_scale, group_rank=c.group_rank)
         else:
             scores, assign, offsets, counts = moe_ops.top_k_gating(logits, c.top_k, renormalize=c.normalize_scores,
                                                                    score_function=c.score_function)
@@ -500,7 +539,8 @@ class DSSandwichRMSNorm(DSPreNormBase):
     """Layers of the form ``x <- x + post_norm(sublayer(pre_norm(x)))`` on an fp32 residual: one kernel closes the
     previous sublayer (``residual += mult * rms_norm(hidden) * gamma_post``; without ``gamma_post`` the sublayer has no
     post-norm: ``residual += mult * hidden``), optionally adds another fp32 stream, and opens the next one (returns
-    ``rms_norm(residual) * gamma``; without ``gamma``: the stream itself in the output dtype if ``copy_out``)."""
+    ``rms_norm(residual) * gamma``; without ``gamma``: the stream itself in the output dtype if ``copy_out``).  Both norms'
+    weights may be stored as their distance from a constant (``gamma_offset``, ``post_offset``)."""
 
     @staticmethod
     def name() -> str:
@@ -511,11 +551,13 @@ class DSSandwichRMSNorm(DSPreNormBase):
         return NormTypeEnum(config.type) == NormTypeEnum.RMSNorm and _dt(config.residual_dtype) == DtypeEnum.fp32
 
     def forward(self, residual, hidden_states, gamma, beta=None, gamma_post=None, extra=None, mult=1.0, copy_out=False,
-                channel_scale=None, gamma_offset=0.0):
+                channel_scale=None, gamma_offset=0.0, post_offset=0.0):
         """``channel_scale`` ``[W]``: what the closed sublayer adds is also multiplied per channel (a layer scale);
-        ``gamma_offset``: the opening norm's weight is ``gamma_offset + gamma`` (1 for weights stored around zero)."""
+        ``gamma_offset`` / ``post_offset``: the opening / closing norm's weight is ``gamma_offset + gamma`` / ``post_offset +
+        gamma_post`` (1 for weights stored around zero)."""
         y = M.resid_norm_step(residual, hidden_states, gamma_post, extra, gamma, self._config.eps,
-                              _dt(self._config.output_dtype).torch, mult, copy_out, channel_scale, gamma_offset)
+                              _dt(self._config.output_dtype).torch, mult, copy_out, channel_scale, gamma_offset,
+                              post_offset)
         return residual, y
 
 
@@ -762,25 +804,7 @@ class DSLatentSinkAttention(DSSelfAttentionBase):
         base = 10000.0 if rot is None else rot.theta_base
         self._inv_freq, self._rot_amp = self.rotary_table(n_rot, base, config.rotary_scaling)
 
-    @staticmethod
-    def rotary_table(n_rot: int, base: float, scaling=None):
-        """fp32 angular frequencies ``base^(-2i / n_rot)`` of the ``n_rot / 2`` pairs and the factor on cos and sin.  With
-        ``scaling``: let ``pair(t) = n_rot ln(original / (2 pi t)) / (2 ln base)`` be the (fractional) pair that makes
-        ``t`` turns over the original context, ``lo = max(floor(pair(fast)), 0)``, ``hi = min(ceil(pair(slow)), n_rot - 1)``
-        and ``w_i = min(1, max(0, (i - lo) / max(hi - lo, 0.001)))``; pair ``i`` turns at ``f_i (1 - w_i) + w_i f_i /
-        factor`` and the amplitude is ``0.1 ln(factor) + 1``.  Evaluated in float64, stored as float32."""
-        i = torch.arange(0, n_rot, 2, dtype=torch.float64) / 2.0
-        f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / max(n_rot, 1))
-        amp = 1.0
-        if scaling is not None and n_rot > 0:
-            def pair(turns: float) -> float:
-                return n_rot * math.log(scaling.original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
-            lo = max(math.floor(pair(scaling.fast)), 0)
-            hi = min(math.ceil(pair(scaling.slow)), n_rot - 1)
-            ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
-            f = f / scaling.factor * ramp + f * (1.0 - ramp)
-            amp = 0.1 * math.log(scaling.factor) + 1.0
-        return f.to(torch.float32), float(amp)
+    rotary_table = staticmethod(scaled_rotary_table)
 
     @property
     def kv_block_size(self) -> int:
@@ -870,10 +894,11 @@ class DSScaledPostRMSNorm(DSPostNormBase):
 
 @DSSelfAttentionRegistry.register_module
 class DSFilteredBiasAttention(DSSelfAttentionBase):
-    """Softmax attention without rotation whose projections pass a short causal filter over time.  Projection columns:
+    """Softmax attention whose projections pass a short causal filter over time.  Projection columns:
     ``q (Hq d) | k (G d) | v (G dv) | gate (Hq dv)``.  Every channel of q | k | v is filtered over the sequence (the last
     ``taps - 1`` projected rows are carried per sequence), q and k heads are RMS-normed with one weight of ``d`` entries
-    each, q is multiplied by ``1 + coef * ln(floor((pos + 1) / every) + 1)``; a key at distance ``n`` behind the query
+    each, q is multiplied by ``1 + coef * ln(floor((pos + 1) / every) + 1)``; the first channels of every q and k head may turn
+    with the position (in either pairing, optionally with :class:`RotaryScalingConfig`), or a key at distance ``n`` behind the query
     adds the learned ``bias[bucket(n), h]`` to its scaled score (buckets: one per distance below half the table's rows,
     logarithmic up to ``far`` above); causal or chunk-local / sliding-window mask; the heads' outputs are multiplied by
     ``sigmoid(gate)``.  Filter sums, norms, temperature, scores, weights and the weighted sum are fp32; the paged cache
@@ -901,7 +926,8 @@ class DSFilteredBiasAttention(DSSelfAttentionBase):
             b = config.distance_bias
             if b is None or b.rows < 2 or b.far <= b.rows // 2:
                 return False
-        elif pe != PositionalEmbeddingType.none:
+        elif pe not in (PositionalEmbeddingType.none, PositionalEmbeddingType.rotate_half,
+                        PositionalEmbeddingType.rotate_every_other):
             return False
         return (config.head_size <= 256 and (config.v_head_size or config.head_size) <= 256
                 and config.n_heads_q % config.n_heads_kv == 0 and 1 <= config.qkv_conv_taps <= 16
@@ -914,6 +940,13 @@ class DSFilteredBiasAttention(DSSelfAttentionBase):
     @property
     def q_block_size(self) -> int:
         return 1
+
+    def __init__(self, config: DSSelfAttentionConfig, implementation_config: Dict[str, Any]) -> None:
+        super().__init__(config, implementation_config)
+        n_rot, base, divisor, self._interleaved = rotated_channels(config)
+        self._inv_freq, self._rot_amp = None, 1.0
+        if n_rot > 0:
+            self._inv_freq, self._rot_amp = scaled_rotary_table(n_rot, base, config.rotary_scaling, divisor)
 
     @property
     def filtered_channels(self) -> int:
@@ -949,9 +982,12 @@ class DSFilteredBiasAttention(DSSelfAttentionBase):
         idx = DSFilteredBiasAttention.bucket_of_distance(table.shape[0], far).to(table.device)
         return table.float().index_select(0, idx).t().contiguous()
 
-    def forward(self, projected: torch.Tensor, kv_cache, batch, inv_freqs=None, weights=None,
-                conv_state=None) -> torch.Tensor:
+    def forward(self, projected: torch.Tensor, kv_cache, batch, inv_freqs=None, weights=None, conv_state=None,
+                out=None, out_scale=1.0) -> torch.Tensor:
+        """``out`` (rows of ``Hq dv`` columns): the result, multiplied by ``out_scale``, goes there."""
         c = self._config
+        if self._inv_freq is not None and self._inv_freq.device != projected.device:
+            self._inv_freq = self._inv_freq.to(projected.device)
         dv = c.v_head_size or c.head_size
         keys, values = kv_cache
         C = self.filtered_channels
@@ -960,7 +996,7 @@ class DSFilteredBiasAttention(DSSelfAttentionBase):
         q = M.qkv_filter_norm_append(projected, conv_w, conv_state, info, weights.q_norm if c.qk_norm_weight else None,
                                      weights.k_norm if c.qk_norm_weight else None, keys, values, t2s, pos, tables,
                                      c.n_heads_q, c.n_heads_kv, c.head_size, dv, c.qk_norm_eps, True, c.q_temp_coef,
-                                     c.q_temp_every)
+                                     c.q_temp_every, self._inv_freq, self._interleaved, self._rot_amp)
         if conv_w is not None and conv_w.shape[1] > 1:
             M.conv_state_update(projected[:, :C], conv_state, info)
         mt = MaskingType(c.masking_type)
@@ -972,7 +1008,7 @@ class DSFilteredBiasAttention(DSSelfAttentionBase):
         bias = weights.dist_bias if c.distance_bias is not None else None
         gate = projected[:, C: C + c.n_heads_q * dv] if c.output_gate else None
         return M.sink_attention(q, keys, values, None, t2s, pos, tables, c.scale_factor, chunk, _dt(c.output_dtype).torch,
-                                atoms, n_long, window=window, dist_bias=bias, gate=gate)
+                                atoms, n_long, window=window, dist_bias=bias, gate=gate, out=out, out_scale=out_scale)
 
 
 @DSSelfAttentionRegistry.register_module
@@ -981,7 +1017,7 @@ class DSRotarySinkAttention(DSSelfAttentionBase):
     (G dv) | gate``, without the v columns when the values are the projected keys themselves (``values_from_keys``: as projected,
     before rotation), the gate (one column per head, or per output channel) starting at the next multiple of 8.  Optional RMS
     norm over the whole q (k) row with a weight per channel (``qk_row_norm``), rotation of the first channels of every head in
-    either pairing with all frequencies divided by one factor, a learned number per query head on the scores, causal /
+    either pairing with all frequencies divided by one factor or slowed by wavelength (``rotary_scaling``), a learned number per query head on the scores, causal /
     chunk-local / sliding-window mask, one added to the softmax denominator (``unit_sink``) or a learned sink logit.  Norms,
     angles, scores, weights and the weighted sum are fp32.
 
@@ -996,7 +1032,7 @@ class DSRotarySinkAttention(DSSelfAttentionBase):
     def supports_config(config: DSSelfAttentionConfig) -> bool:
         if config.kv_latent_dim is not None or config.qkv_conv_taps > 1 or config.q_temp_coef != 0.0:
             return False
-        if config.qk_unit_rms or config.qk_norm_weight or config.rotary_scaling is not None or (config.sink and config.unit_sink):
+        if config.qk_unit_rms or config.qk_norm_weight or (config.sink and config.unit_sink):
             return False
         if MaskingType(config.masking_type) not in (MaskingType.causal, MaskingType.chunked, MaskingType.sliding_window):
             return False
@@ -1011,22 +1047,14 @@ class DSRotarySinkAttention(DSSelfAttentionBase):
 
     def __init__(self, config: DSSelfAttentionConfig, implementation_config: Dict[str, Any]) -> None:
         super().__init__(config, implementation_config)
-        pe, rot = PositionalEmbeddingType(config.positional_embedding_type), config.positional_embedding_config
-        n_rot = 0
-        if pe != PositionalEmbeddingType.none:
-            n_rot = config.head_size if rot is None or rot.rotate_dim is None else rot.rotate_dim
-        if n_rot % 2 or n_rot > config.head_size:
-            raise ValueError(f"cannot rotate {n_rot} of {config.head_size} channels in pairs")
-        self._interleaved = pe == PositionalEmbeddingType.rotate_every_other
-        self._inv_freq = self.rotary_table(n_rot, 10000.0 if rot is None else rot.theta_base,
-                                           1.0 if rot is None else rot.freq_divisor)
+        n_rot, base, divisor, self._interleaved = rotated_channels(config)
+        self._inv_freq, self._rot_amp = scaled_rotary_table(n_rot, base, config.rotary_scaling, divisor)
         self._zero_sink = torch.zeros(config.n_heads_q, dtype=torch.float32) if config.unit_sink else None
 
     @staticmethod
     def rotary_table(n_rot: int, base: float, divisor: float = 1.0) -> torch.Tensor:
         """fp32 angular frequencies ``base^(-2i / n_rot) / divisor`` of the ``n_rot / 2`` pairs, evaluated in float64."""
-        i = torch.arange(0, n_rot, 2, dtype=torch.float64)
-        return (torch.pow(torch.tensor(float(base), dtype=torch.float64), -i / max(n_rot, 1)) / divisor).to(torch.float32)
+        return scaled_rotary_table(n_rot, base, None, divisor)[0]
 
     @property
     def kv_block_size(self) -> int:
@@ -1052,7 +1080,9 @@ class DSRotarySinkAttention(DSSelfAttentionBase):
             n += c.n_heads_kv * (c.v_head_size or c.head_size)
         return (n + 7) // 8 * 8
 
-    def forward(self, projected: torch.Tensor, kv_cache, batch, inv_freqs=None, weights=None) -> torch.Tensor:
+    def forward(self, projected: torch.Tensor, kv_cache, batch, inv_freqs=None, weights=None, out=None,
+                out_scale=1.0) -> torch.Tensor:
+        """``out`` (rows of ``Hq dv`` columns): the result, multiplied by ``out_scale``, goes there."""
         c = self._config
         H, G, d, dv = c.n_heads_q, c.n_heads_kv, c.head_size, c.v_head_size or c.head_size
         keys, values = kv_cache
@@ -1065,7 +1095,7 @@ class DSRotarySinkAttention(DSSelfAttentionBase):
         q = P.rope_append(projected, 0, k0, k0 if c.values_from_keys else k0 + G * d,
                           weights.q_norm if c.qk_row_norm else None, weights.k_norm if c.qk_row_norm else None,
                           self._inv_freq, self._interleaved, weights.q_head_scale if c.q_head_scale else None, keys, values,
-                          t2s, pos, tables, H, G, d, dv, c.qk_norm_eps)
+                          t2s, pos, tables, H, G, d, dv, c.qk_norm_eps, self._rot_amp)
         mt = MaskingType(c.masking_type)
         chunk = int(c.masking_args["size"]) if mt == MaskingType.chunked else 0
         window = int(c.masking_args["size"]) if mt == MaskingType.sliding_window else 0
@@ -1077,7 +1107,7 @@ class DSRotarySinkAttention(DSSelfAttentionBase):
             atoms, n_long = batch.atoms(), batch.atoms_longer_than(M.SHORT_ATOM)
         sink = self._zero_sink if c.unit_sink else (weights.sink if c.sink else None)
         return M.sink_attention(q, keys, values, sink, t2s, pos, tables, c.scale_factor, chunk, _dt(c.output_dtype).torch,
-                                atoms, n_long, window=window, gate=gate)
+                                atoms, n_long, window=window, gate=gate, out=out, out_scale=out_scale)
 
 
 @DSRecurrentMixerRegistry.register_module
@@ -1119,3 +1149,152 @@ class DSRemovalDeltaMixer(_RecurrentMixer):
         o = P.removal_recurrence(buf, S, batch.seq_info(), batch.single_rows())
         return M.group_norm_gate(o, projected[:, 4 * B: 4 * B + H * n], weights.norm, n, c.eps, False,
                                  _dt(c.output_dtype).torch, sigmoid=True)
+
+
+def _column_blocks(*widths: int) -> Tuple[int, ...]:
+    """First column of every block of a fused projection (blocks padded to whole 16-byte words), then the total width."""
+    cols, at = [], 0
+    for w in widths:
+        cols.append(at)
+        at += (w + 7) // 8 * 8
+    return (*cols, at)
+
+
+@DSRecurrentMixerRegistry.register_module
+class DSLightningMixer(_RecurrentMixer):
+    """Lightning attention.  Projection columns (blocks padded to multiples of 8): ``q (H n) | k (H n) | v (H dv) | g (H dv)``; q, k
+    and v pass a SiLU; per head ``S <- decay_h S + k v^T``, ``o = S^T q`` with the fixed ``head_decay``; the output is ``o / rms(o) *
+    norm * sigmoid(g)`` with one rms over all heads.  ``weights``: ``norm`` ``[H dv]``."""
+
+    @staticmethod
+    def name() -> str:
+        return "lightning_mixer"
+
+    @staticmethod
+    def supports_config(config: DSRecurrentMixerConfig) -> bool:
+        return (config.kind == "lightning" and config.key_dim <= 256 and config.n_heads == config.n_heads_kv
+                and config.head_decay is not None and len(config.head_decay) == config.n_heads)
+
+    def __init__(self, config, implementation_config):
+        super().__init__(config, implementation_config)
+        self._decay = torch.tensor(config.head_decay, dtype=torch.float32)
+
+    @property
+    def output_width(self) -> int:
+        return self._config.n_heads * self._config.value_dim
+
+    @property
+    def columns(self) -> Tuple[int, ...]:
+        c = self._config
+        return _column_blocks(c.n_heads * c.key_dim, c.n_heads * c.key_dim, self.output_width, self.output_width)
+
+    @property
+    def projection_width(self) -> int:
+        return self.columns[-1]
+
+    def state_shapes(self):
+        c = self._config
+        return [((c.n_heads, c.value_dim, c.key_dim), torch.float32)]
+
+    def forward(self, projected, weights, states, batch, out=None, out_scale=1.0):
+        c = self._config
+        H, n, dv = c.n_heads, c.key_dim, c.value_dim
+        (S,) = states
+        if self._decay.device != projected.device:
+            self._decay = self._decay.to(projected.device)
+        q0, k0, v0, g0, _ = self.columns
+        x = Gt.silu_columns(projected[:, :g0])
+        o = M.linear_recurrence(x[:, k0: k0 + H * n], x[:, q0: q0 + H * n], x[:, v0: v0 + H * dv], self._decay, None, None, S,
+                                batch.seq_info(), H, H, n, dv, False)
+        return M.group_norm_gate(o, projected[:, g0: g0 + H * dv], weights.norm, H * dv, c.eps, False, _dt(c.output_dtype).torch,
+                                 sigmoid=True, out=out, out_scale=out_scale)
+
+
+@DSRecurrentMixerRegistry.register_module
+class DSGatedLinearMixer(_RecurrentMixer):
+    """Gated linear attention.  Projection columns (blocks padded to multiples of 8): ``q (H n) | k (H n) | v (H dv) | g (H dv) | low
+    (rank)``; per head ``S <- diag(decay) S + k v^T``, ``o = S^T q`` with ``q`` scaled by ``n^-1/2`` and ``decay = sigmoid(low w2 +
+    bias)^(1 / decay_tau)`` per key channel; the output is ``o / rms(o) * norm * silu(g)`` per head.  ``weights``: ``w2`` ``[rank,
+    H n]``, ``decay_bias`` fp32 ``[H n]``, ``norm`` ``[dv]``."""
+
+    @staticmethod
+    def name() -> str:
+        return "gated_linear_mixer"
+
+    @staticmethod
+    def supports_config(config: DSRecurrentMixerConfig) -> bool:
+        return (config.kind == "channel_decay" and config.key_dim <= 256 and config.n_heads == config.n_heads_kv
+                and config.decay_tau > 0.0)
+
+    @property
+    def output_width(self) -> int:
+        return self._config.n_heads * self._config.value_dim
+
+    @property
+    def columns(self) -> Tuple[int, ...]:
+        """First columns of q, k, v, g and low."""
+        c = self._config
+        return _column_blocks(c.n_heads * c.key_dim, c.n_heads * c.key_dim, self.output_width, self.output_width)
+
+    def state_shapes(self):
+        c = self._config
+        return [((c.n_heads, c.value_dim, c.key_dim), torch.float32)]
+
+    def forward(self, projected, weights, states, batch, out=None, out_scale=1.0):
+        c = self._config
+        H, n, dv = c.n_heads, c.key_dim, c.value_dim
+        (S,) = states
+        q0, k0, v0, g0, low0 = self.columns
+        x, decay = Gt.decay_prepare(projected, q0, k0, v0, low0, weights.w2, weights.decay_bias, H * n, H * dv, n ** -0.5,
+                                    c.decay_tau)
+        o = M.linear_recurrence(x[:, H * n: 2 * H * n], x[:, : H * n], x[:, 2 * H * n:], decay, None, None, S, batch.seq_info(),
+                                H, H, n, dv, False)
+        return M.group_norm_gate(o, projected[:, g0: g0 + H * dv], weights.norm, dv, c.eps, False, _dt(c.output_dtype).torch,
+                                 out=out, out_scale=out_scale)
+
+
+@DSRecurrentMixerRegistry.register_module
+class DSLinearRecurrentUnit(_RecurrentMixer):
+    """Gated linear recurrent unit of ``N = n_heads * key_dim`` channels in ``n_heads`` blocks.  Projection columns (blocks padded to
+    multiples of 8): ``y (N) | x (N)``.  ``u = filter(x + x_bias) + conv_b``; per block ``r, i = sigmoid(u_b W + bias)``; ``log a = r *
+    rate`` with ``rate = -decay_rate softplus(lam)``; ``s <- a s + sqrt(1 - a^2) i u``; the output is ``s * gelu(y + y_bias)``.
+    ``weights``: ``conv_w`` ``[N, taps]``, ``conv_b``, ``x_bias``, ``y_bias`` ``[N]``, ``gate_w`` ``[2, n_heads, key_dim (in), key_dim
+    (out)]``, ``gate_b`` fp32 ``[2, N]``, ``rate`` fp32 ``[N]``."""
+
+    @staticmethod
+    def name() -> str:
+        return "linear_recurrent_unit"
+
+    @staticmethod
+    def supports_config(config: DSRecurrentMixerConfig) -> bool:
+        return config.kind == "lru" and 1 <= config.conv_taps <= 16 and config.decay_rate > 0.0
+
+    @property
+    def output_width(self) -> int:
+        return self._config.n_heads * self._config.key_dim
+
+    @property
+    def columns(self) -> Tuple[int, ...]:
+        return _column_blocks(self.output_width, self.output_width)
+
+    @property
+    def projection_width(self) -> int:
+        return self.columns[-1]
+
+    def state_shapes(self):
+        """The channels' states, then the filter's carried inputs (none for a single tap)."""
+        c, N = self._config, self.output_width
+        shapes = [((N,), torch.float32)]
+        if c.conv_taps > 1:
+            shapes.append(((c.conv_taps - 1, N), _dt(c.input_dtype).torch))
+        return shapes
+
+    def forward(self, projected, weights, states, batch, out=None, out_scale=1.0):
+        N = self.output_width
+        s, conv_state = states[0], states[1] if len(states) > 1 else None
+        y0, x0, _ = self.columns
+        y, x = projected[:, y0: y0 + N], projected[:, x0: x0 + N]
+        info = batch.seq_info()
+        u = M.conv_silu(x, weights.conv_w, weights.conv_b, conv_state, info, batch.token_to_seq(), weights.x_bias, act=False)
+        a, g = Gt.lru_gates(u, weights.gate_w, weights.gate_b, weights.rate)
+        return Gt.lru_scan(a, g, y, weights.y_bias, x, s, conv_state, info, batch.single_rows(), out, out_scale)

@@ -17,7 +17,7 @@ from ..native import lib as _lib
 
 _lib.register({
     "sxb_top_k_gating": "ppppp" "iiii" "i" "p",
-    "sxb_grouped_top_k_gating": "pppppp" "iiiii" "f" "p",
+    "sxb_grouped_top_k_gating": "pppppp" "iiiii" "f" "i" "p",
     "sxb_copy_group_rows": "ppp" "iii" "l" "p",
     "sxb_moe_scatter": "ppppppp" "iiiii" "p",
     "sxb_moe_scatter_scaled": "pppppppp" "iiiii" "p",
@@ -27,16 +27,18 @@ _lib.register({
 
 
 def top_k_gating(logits: torch.Tensor, top_k: int, renormalize: bool = True, score_function: str = "softmax",
-                 correction: torch.Tensor = None, n_groups: int = 1, keep_groups: int = 1, scale: float = 1.0):
+                 correction: torch.Tensor = None, n_groups: int = 1, keep_groups: int = 1, scale: float = 1.0,
+                 group_rank: str = "max"):
     """``logits`` [T, E] -> ``(scores fp32 [T,K], assignments int32 [T,K], offsets int32 [T,K], counts int32 [E])``.
 
     ``score_function`` ``"softmax"``: scores are the softmax over all experts; ``"sigmoid"``: every expert is scored on
     its own with ``sigmoid(logit)``.  The ``top_k`` largest win either way; ``renormalize`` divides them by their sum.
 
-    Group-limited choice (softmax scores only; taken when ``correction`` is given, ``n_groups > 1`` or ``scale != 1``):
-    the winners are the ``top_k`` largest ``score + correction`` (``correction`` fp32 ``[E]``) among the experts of the
-    ``keep_groups`` groups -- of ``n_groups`` equal contiguous blocks of experts -- whose best ``score + correction``
-    is largest; the returned scores are the winners' plain scores normalised by their total (1e-20 added), times ``scale``.
+    Group-limited choice (taken when ``correction`` is given, ``n_groups > 1`` or ``scale != 1``): the winners are the
+    ``top_k`` largest ``score + correction`` (``correction`` fp32 ``[E]``) among the experts of the ``keep_groups`` groups
+    -- of ``n_groups`` equal contiguous blocks of experts -- that rank first: by their best ``score + correction``
+    (``group_rank`` ``"max"``) or by the sum of their two best (``"top2"``); the returned scores are the winners' plain
+    scores, with ``renormalize`` divided by their total (1e-20 added), times ``scale``.
 
     ``offsets[t,k]`` is the arrival index of token ``t`` inside expert ``assignments[t,k]`` (a permutation of
     ``range(counts[e])`` per expert; on CUDA the order is nondeterministic, on CPU it is token order)."""
@@ -50,8 +52,8 @@ def top_k_gating(logits: torch.Tensor, top_k: int, renormalize: bool = True, sco
     counts = torch.empty(E, dtype=torch.int32, device=dev)
     grouped = correction is not None or n_groups > 1 or scale != 1.0
     if grouped:
-        if score_function != "softmax":
-            raise ValueError("the group-limited choice scores with the softmax over all experts")
+        if group_rank not in ("max", "top2"):
+            raise ValueError(f"unknown group rank {group_rank!r}")
         if E % n_groups or not 1 <= keep_groups <= n_groups or top_k > keep_groups * (E // n_groups):
             raise ValueError(f"cannot choose {top_k} of {E} experts in {keep_groups} of {n_groups} groups")
     if grouped and logits.is_cuda:
@@ -59,20 +61,21 @@ def top_k_gating(logits: torch.Tensor, top_k: int, renormalize: bool = True, sco
         corr = None if correction is None else correction.float().contiguous()
         _lib.call("sxb_grouped_top_k_gating", logits.data_ptr(), _lib.ptr(corr), scores.data_ptr(), assign.data_ptr(),
                   offsets.data_ptr(), counts.data_ptr(), T, E, top_k, int(n_groups), int(keep_groups), float(scale),
+                  (1 if score_function == "sigmoid" else 0) | (2 if group_rank == "top2" else 0) | (0 if renormalize else 4),
                   _lib.stream_ptr())
         return scores, assign, offsets, counts
     if grouped:
-        probs = torch.softmax(logits.float(), dim=-1)
+        probs = torch.sigmoid(logits.float()) if score_function == "sigmoid" else torch.softmax(logits.float(), dim=-1)
         choice = probs if correction is None else probs + correction.float()
         if keep_groups < n_groups:
             per = E // n_groups
-            best = choice.view(T, n_groups, per).max(dim=-1).values
+            best = choice.view(T, n_groups, per).topk(min(per, 2 if group_rank == "top2" else 1), dim=-1).values.sum(dim=-1)
             kept = torch.zeros(T, n_groups, dtype=torch.bool, device=dev)
             kept.scatter_(1, torch.topk(best, keep_groups, dim=-1).indices, True)
             choice = choice.masked_fill(~kept.repeat_interleave(per, dim=1), float("-inf"))
         a = torch.topk(choice, top_k, dim=-1).indices
         s = probs.gather(1, a)
-        s = s / (s.sum(dim=-1, keepdim=True) + 1e-20) * scale
+        s = (s / (s.sum(dim=-1, keepdim=True) + 1e-20) if renormalize else s) * scale
         flat = a.reshape(-1)
         onehot = torch.nn.functional.one_hot(flat, E)
         order = (torch.cumsum(onehot, dim=0) - 1).gather(1, flat[:, None]).squeeze(1)
