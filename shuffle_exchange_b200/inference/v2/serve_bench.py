@@ -10,7 +10,9 @@ shared expert, per-layer token input) next to a Fomalix stack of attention layer
 with a decay per key channel, three-power dense feed-forward, clamped experts chosen among groups with identity experts)
 next to the Kekopel stack of equal size whose window holds every key.  With ``--serve-model vezodra`` the pair is a Vezodra
 stack (mixer and feed-forward of one stream, rotary attention, windowed attention beside a delta rule with removal and decay
-vectors) next to a Fomalix stack of attention and delta-rule layers of equal size.
+vectors) next to a Fomalix stack of attention and delta-rule layers of equal size.  With ``--serve-model sudupel`` the pair is
+a Sudupel stack (lightning attention, windowed attention beside gated linear attention, sink attention beside a gated linear
+recurrent unit) next to the Vezodra stack of equal size.
 
 Timing: CUDA events on the launching stream, >= 3 warm-up forwards, a buffer larger than L2 is rewritten between timed
 forwards.  Prefill: one request of ``prefill`` tokens in one forward.  Decode: ``batch`` requests with ``context`` tokens
@@ -1128,6 +1130,277 @@ def vezodra_kernel_table(z: Dict, prefill: int, batch: int, context: int, timer,
     return rows
 
 
+# ------------------------------------------------------------------------------------------------ Sudupel beside Vezodra
+SUDUPEL = dict(taps=4, rank=16, lru_taps=4, block=256, experts=8, groups=2, keep=1, top=2, limit=7.0, tau=16.0,
+               yarn=dict(factor=4.0, original=2048, fast=32.0, slow=1.0))
+
+
+def sudupel_config(z: Dict) -> Dict:
+    """Layers cycle lightning / windowed attention beside gated linear attention / attention beside the recurrent unit (as wide as
+    the stream); feed-forwards are dense except for every fourth layer's experts of a quarter of the width."""
+    d, H, G, W = z["head"], z["heads"], z["kv_heads"], z["width"]
+    att = {"dim": d, "heads": H, "kv_heads": G, "scale": d ** -0.5, "vdim": d}
+    kinds = [
+        ("lightning", {"dim": d, "heads": H, "vdim": d, "decay": [1.0 - 2.0 ** (-2.0 - 6.0 * h / H) for h in range(H)]}),
+        ("parallel_2", {"left": dict(att, conv=SUDUPEL["taps"], mask={"size": WINDOW}, rot={"base": 10000.0, "dims": d}),
+                        "right": {"dim": d, "heads": H, "vdim": d, "tau": SUDUPEL["tau"]}, "left_scale": 0.7, "right_scale": 0.6}),
+        ("parallel", {"left": dict(att, rot={"base": 10000.0, "dims": d, "scaling": SUDUPEL["yarn"]}),
+                      "right": {"width": W, "blocks": max(1, W // SUDUPEL["block"]), "conv": SUDUPEL["lru_taps"]},
+                      "left_scale": 0.7, "right_scale": 0.6}),
+    ]
+    dense = {"ff": z["ff"], "kind": "dense", "limit": SUDUPEL["limit"]}
+    moe = {"expert": {"ff": z["ff"] // 4}, "kind": "moe",
+           "router": {"experts": SUDUPEL["experts"], "groups": {"count": SUDUPEL["groups"], "keep": SUDUPEL["keep"]},
+                      "top": SUDUPEL["top"]}}
+    layers = [{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1], "mlp": moe if i % 4 == 1 else dense}
+              for i in range(z["layers"])]
+    return {"architecture": "Sudupel", "embedding": {"scale": 1.0}, "layers": layers, "logit_softcap": 30.0,
+            "norm": {"eps": 1e-5}, "vocab": VOCAB, "width": W}
+
+
+def sudupel_weights(cfg: Dict, device) -> Dict[str, torch.Tensor]:
+    g = torch.Generator(device=device).manual_seed(0)
+    W, bf, rk = cfg["width"], torch.bfloat16, SUDUPEL["rank"]
+
+    def mat(*shape):
+        return (torch.randn(*shape, generator=g, device=device) / math.sqrt(shape[-1])).to(bf)
+
+    def vec(n, lo=0.5, hi=1.5):
+        return (torch.rand(n, generator=g, device=device) * (hi - lo) + lo).to(bf)
+
+    out = {"embed": mat(cfg["vocab"], W), "head": mat(cfg["vocab"], W), "final.norm": vec(W, -0.3, 0.3)}
+    for i, L in enumerate(cfg["layers"]):
+        m, p = L["mixer"], f"l{i}."
+        for n in ("norm1", "norm1b", "norm2", "norm2b"):
+            out[p + n] = vec(W, -0.3, 0.3)
+        if L["type"] == "lightning":
+            H, n, dv = m["heads"], m["dim"], m["vdim"]
+            for name, o in (("q", H * n), ("k", H * n), ("v", H * dv), ("g", H * dv)):
+                out[p + "mix." + name] = mat(o, W)
+            out[p + "mix.norm"], out[p + "mix.o"] = vec(H * dv), mat(W, H * dv)
+        else:
+            a, b, q = m["left"], m["right"], p + "mix.left."
+            H, G, d, dv = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            whole = L["type"] == "parallel"
+            for name, o in (("q", H * d), ("k", G * d), ("v", G * dv)):
+                out[q + name] = mat(o, W)
+                if not whole:
+                    out[q + name + ".conv"] = vec(o * a["conv"], -0.5, 0.5).view(o, a["conv"])
+            out[q + "q.norm"], out[q + "k.norm"] = vec(H * d if whole else d), vec(G * d if whole else d)
+            out[q + "o"], q = mat(W, H * dv), p + "mix.right."
+            if whole:
+                N, B = b["width"], b["blocks"]
+                for name in ("y", "x"):
+                    out[q + name], out[q + name + ".b"] = mat(N, W), vec(N, -0.1, 0.1)
+                out[q + "conv"], out[q + "conv.b"] = vec(N * b["conv"], -0.5, 0.5).view(N, b["conv"]), vec(N, -0.1, 0.1)
+                for name in ("ra", "ri"):
+                    out[q + name], out[q + name + ".b"] = mat(B, N // B, N // B), vec(N, -1, 1).view(B, N // B)
+                out[q + "lam"], out[q + "o"] = vec(N, -6, -2), mat(W, N)
+            else:
+                H, n, dv = b["heads"], b["dim"], b["vdim"]
+                for name, o in (("q", H * n), ("k", H * n), ("v", H * dv), ("g", H * dv)):
+                    out[q + name] = mat(o, W)
+                out[q + "a1"], out[q + "a2"], out[q + "a2.b"] = mat(rk, W), mat(H * n, rk), vec(H * n, 0, 3)
+                out[q + "norm"], out[q + "o"] = vec(dv), mat(W, H * dv)
+        mlp = L["mlp"]
+        if mlp["kind"] == "dense":
+            ff = mlp["ff"]
+            out[p + "mlp.gate"], out[p + "mlp.up"], out[p + "mlp.down"] = mat(ff, W), mat(ff, W), mat(W, ff)
+        else:
+            F_, E = mlp["expert"]["ff"], mlp["router"]["experts"]
+            out[p + "mlp.router"], out[p + "mlp.correction"] = mat(E, W), vec(E, -0.05, 0.05)
+            for e in range(E):
+                out[p + f"mlp.e{e}.gate"], out[p + f"mlp.e{e}.up"] = mat(F_, W), mat(F_, W)
+                out[p + f"mlp.e{e}.down"] = mat(W, F_)
+    return out
+
+
+def build_sudupel(z: Dict, max_tokens: int, max_seqs: int, pages: int):
+    cfg = sudupel_config(z)
+    return build_engine_from_state_dict(cfg, sudupel_weights(cfg, "cuda"), _engine_config(max_tokens, max_seqs, pages),
+                                        dtype=torch.bfloat16)
+
+
+def sudupel_kernel_table(z: Dict, prefill: int, batch: int, context: int, timer, hbm_gbs: float,
+                         peak_tflops: Dict[str, float]) -> List[Dict]:
+    """Every kernel the Sudupel stack adds or takes in a new form, beside the kernel of the Vezodra (or another hybrid) stack that
+    does the like job (``like``), at prefill (one request) and decode (``batch`` requests) shapes: device time, algorithmic
+    bytes and FLOPs, fraction of the roofline (the larger of bytes / copy bandwidth and FLOPs / the peak of the unit used)."""
+    from ...ops import functional as F
+    from ...ops import moe_ops
+    from .kernels import gated_ops as Gt
+    from .kernels import mixer_ops as M
+    from .kernels import parallel_ops as P
+    from .modules.configs import RotaryScalingConfig
+    from .modules.implementations import scaled_rotary_table
+    from .ragged.ragged_wrapper import RaggedBatchWrapper
+    dev, bf = "cuda", torch.bfloat16
+    W, H, G, d, ff, taps, rk = z["width"], z["heads"], z["kv_heads"], z["head"], z["ff"], SUDUPEL["taps"], SUDUPEL["rank"]
+    n = H * d
+    rows: List[Dict] = []
+
+    def add(name, like, phase, fn, nbytes, flops=0.0, pipe=None):
+        ms = timer(fn, 5, 3)
+        ideal_ms = nbytes / hbm_gbs / 1e6
+        if pipe is not None:
+            ideal_ms = max(ideal_ms, flops / peak_tflops[pipe] / 1e9)
+        rows.append({"kernel": name, "like": like, "phase": phase, "ms": round(ms, 4),
+                     "GB_s": round(nbytes / ms / 1e6, 1), "GFLOP_s": round(flops / ms / 1e6, 1), "pipe": pipe or "memory",
+                     "of_roofline": round(ideal_ms / ms, 3)})
+
+    def randn(*shape, dtype=torch.float32):
+        return torch.randn(*shape, device=dev).to(dtype)
+
+    for phase, T, n_seq, seen in (("prefill", prefill, 1, 0), ("decode", batch, batch, context)):
+        per = T // n_seq
+        tot = seen + per
+        n_pages_seq = (tot + 63) // 64
+        t2s = torch.arange(n_seq, device=dev, dtype=torch.int32).repeat_interleave(per)
+        pos = (torch.arange(per, device=dev, dtype=torch.int32) + seen).repeat(n_seq)
+        tables = torch.arange(n_seq * n_pages_seq, device=dev, dtype=torch.int32).view(n_seq, n_pages_seq)
+        info = torch.tensor([[i * per, per, seen, i] for i in range(n_seq)], dtype=torch.int32, device=dev)
+        single = per == 1
+        # closing a sublayer and opening the next
+        x32, y, a = randn(T, W), randn(T, W, dtype=bf), randn(T, W, dtype=bf)
+        wv = torch.zeros(W, device=dev, dtype=bf)
+        mine = "resid_norm_step (both norms' weights around zero)"
+        add(mine, None, phase,
+            lambda: M.resid_norm_step(x32, y, wv, None, wv, 1e-5, bf, w_add=1.0, post_add=1.0), T * W * (4 + 4 + 2 + 2))
+        add("llama rms_norm with residual add", mine, phase, lambda: F.rms_norm(y, wv, 1e-5, a), T * W * 2 * 4)
+        # attention rows
+        C = (H + 2 * G) * d
+        wide = randn(T, C, dtype=bf)
+        inv, amp = scaled_rotary_table(d, 10000.0, RotaryScalingConfig(**SUDUPEL["yarn"]))
+        inv = inv.to(dev)
+        kc, vc = randn(n_seq * n_pages_seq, 64, G, d, dtype=bf), randn(n_seq * n_pages_seq, 64, G, d, dtype=bf)
+        qn, kn, hn = torch.ones(n, device=dev, dtype=bf), torch.ones(G * d, device=dev, dtype=bf), torch.ones(d, device=dev, dtype=bf)
+        row_bytes = T * (n * 6 + 2 * G * d * 4)
+        mine = "rope_append (whole-row norms, halves, amplitude)"
+        add(mine, None, phase,
+            lambda: P.rope_append(wide, 0, n, n + G * d, qn, kn, inv, False, None, kc, vc, t2s, pos, tables, H, G, d, d, 1e-5, amp),
+            row_bytes)
+        add("rope_append (whole-row norms, halves)", mine, phase,
+            lambda: P.rope_append(wide, 0, n, n + G * d, qn, kn, inv, False, None, kc, vc, t2s, pos, tables, H, G, d, d, 1e-5),
+            row_bytes)
+        cw, cst = randn(C, taps, dtype=bf), torch.zeros(n_seq, taps - 1, C, device=dev, dtype=bf)
+        fb = row_bytes + n_seq * (taps - 1) * C * 2 * (2 if seen else 1)
+
+        def filtered(freq):
+            M.qkv_filter_norm_append(wide, cw, cst, info, hn, hn, kc, vc, t2s, pos, tables, H, G, d, d, 1e-5, True, inv_freq=freq)
+            M.conv_state_update(wide, cst, info)
+        mine = "qkv_filter_norm_append (per-head norms, rotation) + state update"
+        add(mine, None, phase, lambda: filtered(inv), fb)
+        add("qkv_filter_norm_append (per-head norms) + state update", mine, phase, lambda: filtered(None), fb)
+        # attention into one half of the pair's output rows
+        wrap = RaggedBatchWrapper(max(T, 64), n_seq, n_pages_seq, device=dev)
+
+        class _Seq:
+            def __init__(self, i):
+                self.seen_tokens, self._b = seen, tables[i].cpu()
+
+            def kv_blocks(self):
+                return self._b
+        for i in range(n_seq):
+            wrap.insert_sequence(_Seq(i), torch.zeros(per, dtype=torch.int32), do_checks=False)
+        wrap.finalize()
+        atoms, n_long = wrap.atoms(), wrap.atoms_longer_than(M.SHORT_ATOM)
+        q32, sink, both = randn(T, H, d), torch.zeros(H, device=dev), torch.empty(T, 2 * n, device=dev, dtype=bf)
+        keys_per_q = (per + 1) / 2 if phase == "prefill" else tot
+        att_bytes, fl = n_seq * tot * 2 * G * d * 2 + T * H * d * 6, 4.0 * T * H * d * keys_per_q
+        gate = randn(T, 8 * ((H + 7) // 8), dtype=bf)
+
+        def attend(sink=None, **kw):
+            return M.sink_attention(q32, kc, vc, sink, t2s, pos, tables, d ** -0.5, 0, bf, atoms, n_long, **kw)
+        mine = "sink_attention (causal, added one, scaled into a column slice)"
+        add(mine, None, phase, lambda: attend(sink, out=both[:, :n], out_scale=0.7), att_bytes, fl, "fp32")
+        add("sink_attention (causal, added one, gate per head)", mine, phase, lambda: attend(sink, gate=gate[:, :H]), att_bytes, fl,
+            "fp32")
+        mine = f"sink_attention (window {tot}, scaled into a column slice)"
+        add(mine, None, phase, lambda: attend(window=tot, out=both[:, :n], out_scale=0.7), att_bytes, fl, "fp32")
+        add(f"sink_attention (window {tot})", mine, phase, lambda: attend(window=tot), att_bytes, fl, "fp32")
+        # matrix states: operands, recurrences, output norms
+        proj = randn(T, 5 * n + 8 * ((rk + 7) // 8), dtype=bf)
+        add("silu_columns (q, k, v)", None, phase, lambda: Gt.silu_columns(proj[:, : 3 * n]), T * 3 * n * 6)
+        add("mlstm_prepare (q, k, v)", "silu_columns (q, k, v)", phase, lambda: M.mlstm_prepare(proj, H, d, d, 1.0), T * 3 * n * 6)
+        w2, zero = randn(rk, n, dtype=bf), torch.zeros(n, device=dev)
+        mine = "decay_prepare (q, k, v, decay per key channel; inner projection)"
+        add(mine, None, phase, lambda: Gt.decay_prepare(proj, 0, n, 2 * n, 5 * n, w2, zero, n, n, 0.1, 16.0),
+            T * (n * (3 * 2 + 4 * 4) + rk * 2) + rk * n * 2, 2.0 * T * n * rk, "fp32")
+        add("removal_prepare (same inner size)", mine, phase,
+            lambda: P.removal_prepare(proj, 0, n, 2 * n, 3 * n, 5 * n, w2, zero, zero, H, d, 0.6, 1e-6),
+            T * (n * (4 * 2 + 5 * 4) + rk * 2) + rk * n * 2, 2.0 * T * n * rk, "fp32")
+        xs = randn(T, 3 * n)
+        xs[:, : 2 * n] /= math.sqrt(d)
+        fixed, per_row = torch.rand(H, device=dev) * 0.1 + 0.9, torch.rand(T, H, device=dev) * 0.1 + 0.9
+        chan, beta = torch.rand(T, n, device=dev) * 0.1 + 0.9, torch.rand(T, H, device=dev)
+        S0 = torch.zeros(n_seq, H, d, d, device=dev)
+        sb = n_seq * H * d * d * 4 * (2 if seen else 1)
+
+        def recur(decay, b, delta):
+            return M.linear_recurrence(xs[:, n: 2 * n], xs[:, :n], xs[:, 2 * n:], decay, b, None, S0, info, H, H, d, d, delta)
+        add("linear_recurrence (fixed decay per head)", None, phase, lambda: recur(fixed, None, False), sb + T * n * 4 * 4,
+            4.0 * T * n * d, "fp32")
+        add("linear_recurrence (delta, decay per head)", "linear_recurrence (fixed decay per head)", phase,
+            lambda: recur(per_row, beta, True), sb + T * n * 4 * 4, 6.0 * T * n * d, "fp32")
+        add("linear_recurrence (decay per key channel)", None, phase, lambda: recur(chan, None, False), sb + T * n * 5 * 4,
+            5.0 * T * n * d, "fp32")
+        buf = P.removal_prepare(proj, 0, n, 2 * n, 3 * n, 5 * n, w2, zero, zero, H, d, 0.6, 1e-6)
+        add("removal_recurrence", "linear_recurrence (decay per key channel)", phase,
+            lambda: P.removal_recurrence(buf, S0, info, single), sb + T * n * (5 + 1) * 4, 9.0 * T * n * d, "fp32")
+        o0, gt = randn(T, n), randn(T, n, dtype=bf)
+        add("group_norm_gate (whole row, sigmoid gate)", None, phase,
+            lambda: M.group_norm_gate(o0, gt, qn, n, 1e-5, False, bf, sigmoid=True), T * n * 8)
+        add("group_norm_gate (per head, silu gate, scaled into a column slice)", None, phase,
+            lambda: M.group_norm_gate(o0, gt, hn, d, 1e-5, False, bf, out=both[:, n:], out_scale=0.6), T * n * 8)
+        for mine in ("group_norm_gate (whole row, sigmoid gate)",
+                     "group_norm_gate (per head, silu gate, scaled into a column slice)"):
+            add("group_norm_gate (per head, sigmoid gate)", mine, phase,
+                lambda: M.group_norm_gate(o0, gt, qn, d, 1e-5, False, bf, sigmoid=True), T * n * 8)
+        # recurrent unit as wide as the stream
+        N, B, lt = W, max(1, W // SUDUPEL["block"]), SUDUPEL["lru_taps"]
+        yx = randn(T, 2 * N, dtype=bf)
+        lcw, lb, lst = randn(N, lt, dtype=bf), torch.zeros(N, device=dev, dtype=bf), torch.zeros(n_seq, lt - 1, N, device=dev, dtype=bf)
+        conv_bytes = T * N * 6 + n_seq * (lt - 1) * N * 2
+        add("conv_silu (input bias, no activation)", None, phase,
+            lambda: M.conv_silu(yx[:, N:], lcw, lb, lst, info, t2s, lb, act=False), conv_bytes)
+        add("conv_silu", "conv_silu (input bias, no activation)", phase, lambda: M.conv_silu(yx[:, N:], lcw, lb, lst, info, t2s),
+            conv_bytes)
+        u, gw = randn(T, N), (randn(2, B, N // B, N // B) / math.sqrt(N // B)).to(bf)
+        gb, rate = torch.zeros(2, N, device=dev), -torch.rand(N, device=dev)
+        add("lru_gates", None, phase, lambda: Gt.lru_gates(u, gw, gb, rate), T * N * 12 + gw.numel() * 2, 4.0 * T * N * (N // B), "fp32")
+        add("removal_prepare (same inner size)", "lru_gates", phase,
+            lambda: P.removal_prepare(proj, 0, n, 2 * n, 3 * n, 5 * n, w2, zero, zero, H, d, 0.6, 1e-6),
+            T * (n * (4 * 2 + 5 * 4) + rk * 2) + rk * n * 2, 2.0 * T * n * rk, "fp32")
+        la, lg = Gt.lru_gates(u, gw, gb, rate)
+        ls, lo = torch.zeros(n_seq, N, device=dev), torch.empty(T, n + N, device=dev, dtype=bf)
+        add("lru_scan (gate, state update)", None, phase,
+            lambda: Gt.lru_scan(la, lg, yx[:, :N], lb, yx[:, N:], ls, lst, info, single, lo[:, n:], 0.6),
+            T * N * 12 + n_seq * N * 4 * (2 if seen else 1))
+        ri, rf, hz, hm = gate[:, :H], gate[:, :H], torch.zeros(H, device=dev), torch.zeros(n_seq, H, device=dev)
+        add("mlstm_gate_scan (a scan per head)", "lru_scan (gate, state update)", phase,
+            lambda: M.mlstm_gate_scan(ri, rf, hz, hz, 15.0, hm, info), T * H * (2 * 2 + 3 * 4) + n_seq * H * 8)
+        # feed-forwards
+        hg = randn(T, 2 * ff, dtype=bf)
+        add("gated_act_rows (clamped)", None, phase, lambda: M.gated_act_rows(hg, "clamped_swish", 7.0), T * ff * 6)
+        add("gated_act (silu)", "gated_act_rows (clamped)", phase, lambda: F.gated_act(hg, "silu"), T * ff * 6)
+        E, K = SUDUPEL["experts"], SUDUPEL["top"]
+        logits, corr = randn(T, E), torch.zeros(E, device=dev)
+        mine = "grouped_top_k_gating (sigmoid, two best, plain weights)"
+        add(mine, None, phase,
+            lambda: moe_ops.top_k_gating(logits, K, renormalize=False, score_function="sigmoid", correction=corr,
+                                         n_groups=SUDUPEL["groups"], keep_groups=SUDUPEL["keep"], group_rank="top2"),
+            T * (E * 4 + K * 12))
+        add("grouped_top_k_gating (softmax, best)", mine, phase,
+            lambda: moe_ops.top_k_gating(logits, K, correction=corr, n_groups=SUDUPEL["groups"], keep_groups=SUDUPEL["keep"]),
+            T * (E * 4 + K * 12))
+    by_name = {(r_["kernel"], r_["phase"]): r_ for r_ in rows}
+    for r_ in rows:                      # distance from the roofline relative to the like kernel's
+        if r_["like"]:
+            mine = by_name[(r_["like"], r_["phase"])]
+            mine["like_of_roofline"], mine["like_kernel"] = r_["of_roofline"], r_["kernel"]
+    return rows
+
+
 def run(sizes: List[str], prefill: int, batch: int, context: int, steps: int, warmup: int, kernels: bool = True,
         chunk: int = 0, model: str = "fomalix") -> Dict:
     global CHUNK, WINDOW
@@ -1190,6 +1463,20 @@ def run(sizes: List[str], prefill: int, batch: int, context: int, steps: int, wa
                                                                   warmup, timer)}
             if kernels:
                 entry["kernels"] = vezodra_kernel_table(z, prefill, batch, context, timer, hbm, peak_tflops)
+            out["sizes"][name] = entry
+        return out
+    if model == "sudupel":
+        out["metric"] = "serving tokens/s, Sudupel vs Vezodra stack of equal size"
+        out["sudupel"], out["vezodra"] = SUDUPEL, VEZODRA
+        WINDOW = CHUNK = max(WINDOW, prefill, context + steps + warmup + 8)    # the windows hold every key: equal work
+        out["attention_window"] = out["attention_chunk"] = WINDOW
+        for name in sizes:
+            z = SIZES[name]
+            entry = {"config": z,
+                     "sudupel": engine_throughput(build_sudupel, z, prefill, batch, context, steps, warmup, timer),
+                     "vezodra": engine_throughput(build_vezodra, z, prefill, batch, context, steps, warmup, timer)}
+            if kernels:
+                entry["kernels"] = sudupel_kernel_table(z, prefill, batch, context, timer, hbm, peak_tflops)
             out["sizes"][name] = entry
         return out
     if model == "ridazen":
